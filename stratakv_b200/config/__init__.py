@@ -5,7 +5,9 @@ from .engine import EngineConfig
 from .fidolix import FidolixConfig
 from .kedelorn import KedelornConfig
 from .povusun import PovusunConfig
+from .tobozen import TobozenConfig
 from .zepavik import ZepavikConfig
 
-__all__ = ["ConfigError", "LlamaConfig", "ZepavikConfig", "PovusunConfig", "KedelornConfig", "FidolixConfig", "EngineConfig", "Architecture", "known_architectures",
+__all__ = ["ConfigError", "LlamaConfig", "ZepavikConfig", "PovusunConfig", "KedelornConfig", "FidolixConfig", "TobozenConfig",
+           "EngineConfig", "Architecture", "known_architectures",
            "load_config", "read_config_json", "register_architecture", "resolve_architecture"]

@@ -126,15 +126,22 @@ __global__ void remember_last_ids_kernel(const int* __restrict__ ids, const int*
 // ---------------------------------------------------------------------------
 // y[r, :] = x[src(r), :] * (1 / sqrt(mean(x^2) + eps)) * gamma, sums in float.
 // The multiplication order is the reference's (src/layers/rmsnorm.cpp:91-93).
+// `groups` > 1: a row is that many equal parts of `hidden` numbers, each divided by its own root mean square; r counts
+// parts, and gamma holds groups * hidden numbers.
 template <typename T>
 __global__ void rmsnorm_kernel(const float* __restrict__ x, const float* __restrict__ gamma,
                                float eps, T* __restrict__ out, const int* __restrict__ rows,
-                               int hidden) {
+                               int hidden, int groups) {
     __shared__ float scratch[33];
     pdl_launch_dependents();
     pdl_wait();
     const int r = blockIdx.x;
-    const int src = rows ? rows[r] : r;
+    int src = rows ? rows[r] : r;
+    if (groups > 1) {
+        const int part = r % groups;
+        src = rows ? rows[r / groups] * groups + part : r;
+        gamma += (size_t)part * hidden;
+    }
     const float* row = x + (size_t)src * hidden;
     float partial = 0.0f;
     for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
@@ -153,12 +160,17 @@ __global__ void rmsnorm_kernel(const float* __restrict__ x, const float* __restr
 template <typename T>
 __global__ void __launch_bounds__(256)
 rmsnorm_rows_kernel(const float* __restrict__ x, const float* __restrict__ gamma, float eps,
-                    T* __restrict__ out, const int* __restrict__ rows, int n_rows, int hidden) {
+                    T* __restrict__ out, const int* __restrict__ rows, int n_rows, int hidden, int groups) {
     pdl_launch_dependents();
     pdl_wait();
     const int r = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (r >= n_rows) return;
-    const int src = rows ? rows[r] : r;
+    int src = rows ? rows[r] : r;
+    if (groups > 1) {
+        const int part = r % groups;
+        src = rows ? rows[r / groups] * groups + part : r;
+        gamma += (size_t)part * hidden;
+    }
     const float4* row = (const float4*)(x + (size_t)src * hidden);
     const int quads = hidden >> 2;
     // The first 2,048 columns of the row stay in registers: all their loads are in flight at once and nothing of
@@ -448,17 +460,20 @@ SKV_EXPORT int skv_embed_sum(const void* table, const void* pair_table, const vo
                       positions, cu_q, slot_ids, last_ids, n_seqs);
 }
 
+// out [n_rows, hidden]; groups: the equal parts of a row that are normed each by itself (1: the whole row).
 SKV_EXPORT int skv_rmsnorm(const float* x, const float* gamma, float eps, void* out, const int* rows,
-                           int n_rows, int hidden, cudaStream_t stream) {
+                           int n_rows, int hidden, int groups, cudaStream_t stream) {
     if (n_rows <= 0) return 0;
-    if (hidden <= 0) return fail("skv_rmsnorm", "hidden must be positive");
+    if (hidden <= 0 || groups <= 0 || hidden % groups) return fail("skv_rmsnorm", "hidden must be positive and split into equal groups");
+    if ((long long)n_rows * groups > 0x7fffffffLL) return fail("skv_rmsnorm", "too many rows");
+    const int parts = n_rows * groups, width = hidden / groups;
     // a warp per row once there are rows enough to fill the GPU that way, else a block per row
-    if (n_rows >= 1024 && hidden % 4 == 0 && (((uintptr_t)x | (uintptr_t)gamma | (uintptr_t)out) & 15) == 0)
-        return launch_pdl("skv_rmsnorm", rmsnorm_rows_kernel<skv_t>, dim3((n_rows + 7) / 8), dim3(256), 0, stream, x,
-                          gamma, eps, (skv_t*)out, rows, n_rows, hidden);
-    const int threads = hidden >= 2048 ? 512 : (hidden >= 512 ? 256 : 128);
-    return launch_pdl("skv_rmsnorm", rmsnorm_kernel<skv_t>, dim3(n_rows), dim3(threads), 0, stream, x, gamma, eps,
-                      (skv_t*)out, rows, hidden);
+    if (parts >= 1024 && width % 4 == 0 && (((uintptr_t)x | (uintptr_t)gamma | (uintptr_t)out) & 15) == 0)
+        return launch_pdl("skv_rmsnorm", rmsnorm_rows_kernel<skv_t>, dim3((parts + 7) / 8), dim3(256), 0, stream, x,
+                          gamma, eps, (skv_t*)out, rows, parts, width, groups);
+    const int threads = width >= 2048 ? 512 : (width >= 512 ? 256 : 128);
+    return launch_pdl("skv_rmsnorm", rmsnorm_kernel<skv_t>, dim3(parts), dim3(threads), 0, stream, x, gamma, eps,
+                      (skv_t*)out, rows, width, groups);
 }
 
 SKV_EXPORT int skv_rope_kv_write(const float* qkv, const float* cos_sin, const int* positions,

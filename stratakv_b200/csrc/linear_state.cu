@@ -1,0 +1,870 @@
+// Linear attention with a matrix state and a decay per head, over packed steps of several sequences: what the mixers of
+// the Mamba-2 and Lightning families have in common, with the steps around it that are theirs alone.
+//
+// A float row holds queries and keys of `groups` heads (dim numbers each) and values of `heads` heads (vdim numbers each);
+// value head h uses query and key head h / (heads / groups).  Per head and position p of a sequence
+//
+//   S_p = exp(l_p) S_(p-1) + c_p k_p v_p^T      (dim x vdim, zero before the first token)
+//   o_p = S_p^T q_p + skip v_p
+//
+// with l_p <= 0 the logarithm of the decay (one number per head, or one per token and head), c_p a factor on the key
+// (or 1) and skip a number per head (or 0).  Queries, keys and values may pass silu as they are read.
+//
+// Everything here is float.  Per sequence the cache keeps S twice, one row per slot [2][heads][dim][vdim]: a step reads
+// the half of the position before its first (by that position's parity) and writes the half of its last, so a one-token
+// step that runs twice (a graph's capture after its warm-up) computes the same thing both times.
+//
+// One token a sequence: one kernel, a block per (head, sequence).  Longer steps: a sequence's tokens are cut into chunks.
+// With S the state before a chunk of L tokens, counted 0 .. L-1 within it,
+//   o_i    = exp(l_0 + .. + l_i) S^T q_i + sum_(j<=i) exp(l_(j+1) + .. + l_i) c_j (q_i . k_j) v_j
+//   S_next = exp(l_0 + .. + l_(L-1)) S + sum_j exp(l_(j+1) + .. + l_(L-1)) c_j k_j v_j^T
+// so a first kernel leaves every chunk's own sum (the second term of S_next) and its decay, a second walks the chunks of
+// a sequence and replaces each sum by the state before its chunk, and a third makes the outputs of all chunks side by
+// side.  The exponents are sums of numbers of one sign, made from the tokens between and never as a difference of two
+// running sums: a token that forgets nearly everything does not cost the tokens after it their precision.
+#include "common.cuh"
+
+namespace skv {
+
+constexpr int LS_THREADS = 256;
+
+struct LinearStateShape {
+    int heads, groups, dim, vdim;
+    int row_stride, q_at, k_at, v_at;      // floats per row, and the columns where queries, keys and values start
+    int silu;                              // queries, keys and values pass silu as they are read
+};
+
+struct LinearStateDecay {
+    const float* decay;                    // [heads]: one decay per head, or null
+    const float* log_decay;                // [tokens][heads]: one logarithm per token and head (decay null)
+    const float* key_scale;                // [tokens][heads] or null
+    const float* skip;                     // [heads] or null
+};
+
+struct LinearStateBatch {
+    const int* positions;                  // [tokens]
+    const int* cu_q;                       // [seqs + 1]
+    const int* slot_ids;                   // [seqs]
+    float* state;                          // [slots][state_stride], S from state_offset on
+    long long state_stride, state_offset;
+};
+
+__device__ __forceinline__ float ls_silu(float z) { return z / (1.0f + expf(-z)); }
+__device__ __forceinline__ float ls_softplus(float z) { return z > 20.0f ? z : log1pf(expf(z)); }
+__device__ __forceinline__ float ls_read(const float* x, int silu) { return silu ? ls_silu(*x) : *x; }
+__device__ __forceinline__ float ls_log(float decay) { return decay > 0.0f ? logf(decay) : -INFINITY; }
+
+// ---- one token a sequence ----------------------------------------------------------------------------------------
+// What the Mamba-2 mixer does between its input projection and the recurrence, for the new token: a causal convolution
+// with bias and silu on the channels [values | keys | queries] (the row's first columns; what lies before the token
+// comes from a ring of the last inputs, row position mod taps), and the step size.
+struct ConvStep {
+    const float* conv_w;                   // [channels][taps], the last column weighs the current token; null: no such step
+    const float* conv_b;                   // [channels]
+    const float* dt_bias;                  // [heads]
+    const float* a_log;                    // [heads]
+    int taps, channels, dt_at;             // dt_at: the column of the row where the step sizes start
+    long long ring_offset;                 // floats from the start of a slot's row: [taps][channels]
+};
+
+__device__ __forceinline__ float conv_one(const float* __restrict__ row, const float* ring, const ConvStep& conv, int p, int c) {
+    float sum = conv.conv_b[c];
+    for (int j = 0; j < conv.taps; ++j) {
+        const int back = conv.taps - 1 - j;
+        if (p - back < 0) continue;
+        const float u = back == 0 ? row[c] : ring[(size_t)((p - back) % conv.taps) * conv.channels + c];
+        sum = fmaf(conv.conv_w[(size_t)c * conv.taps + j], u, sum);
+    }
+    return ls_silu(sum);
+}
+
+// VEC: vdim is a multiple of 4 and a thread takes four neighbouring columns of S; else one column.
+template <int VEC>
+__global__ void __launch_bounds__(LS_THREADS)
+linear_state_step_kernel(const float* __restrict__ rows, float* __restrict__ out, const LinearStateShape shape,
+                         const LinearStateDecay decay, const ConvStep conv, const LinearStateBatch batch) {
+    extern __shared__ __align__(16) float ls_smem[];
+    const int H = shape.heads, N = shape.dim, P = shape.vdim;
+    const int n_pad = (N + 3) & ~3;
+    float* q = ls_smem;                        // [N]
+    float* k = q + n_pad;                      // [N]
+    float* v = k + n_pad;                      // [P rounded up]
+    float* partial = v + ((P + 3) & ~3);       // [LS_THREADS * VEC]
+    __shared__ float head_numbers[2];          // the decay, the skip
+    pdl_launch_dependents();
+    pdl_wait();
+    const int head = blockIdx.x, s = blockIdx.y, g = head / (H / shape.groups);
+    const int t = batch.cu_q[s], p = batch.positions[t];
+    const float* row = rows + (size_t)t * shape.row_stride;
+    float* slot = batch.state + (size_t)batch.slot_ids[s] * batch.state_stride;
+    float scale = 1.0f;
+    if (conv.conv_w) {
+        float* ring = slot + conv.ring_offset;
+        const bool first_of_group = head % (H / shape.groups) == 0;
+        const float dt = ls_softplus(row[conv.dt_at + head] + conv.dt_bias[head]);
+        scale = dt;
+        for (int i = threadIdx.x; i < P + 2 * N; i += LS_THREADS) {
+            const int c = i < P ? shape.v_at + head * P + i
+                                : (i < P + N ? shape.k_at + g * N + i - P : shape.q_at + g * N + i - P - N);
+            const float value = conv_one(row, ring, conv, p, c);
+            if (i < P) v[i] = value;
+            else if (i < P + N) k[i - P] = value * scale;
+            else q[i - P - N] = value;
+            // (the one row of the ring that no tap of this token reads)
+            if (conv.taps > 1 && (i < P || first_of_group)) ring[(size_t)(p % conv.taps) * conv.channels + c] = row[c];
+        }
+        if (threadIdx.x == 0) head_numbers[0] = expf(-expf(conv.a_log[head]) * dt);
+    } else {
+        if (decay.key_scale) scale = decay.key_scale[(size_t)t * H + head];
+        for (int i = threadIdx.x; i < N; i += LS_THREADS) {
+            q[i] = ls_read(row + shape.q_at + g * N + i, shape.silu);
+            k[i] = ls_read(row + shape.k_at + g * N + i, shape.silu) * scale;
+        }
+        for (int i = threadIdx.x; i < P; i += LS_THREADS) v[i] = ls_read(row + shape.v_at + head * P + i, shape.silu);
+        if (threadIdx.x == 0) head_numbers[0] = decay.decay ? decay.decay[head] : expf(decay.log_decay[(size_t)t * H + head]);
+    }
+    if (threadIdx.x == 1) head_numbers[1] = decay.skip ? decay.skip[head] : 0.0f;
+    __syncthreads();
+    const float a = head_numbers[0];
+    const size_t half_size = (size_t)H * N * P;
+    const float* __restrict__ before = slot + batch.state_offset + (size_t)((p - 1) & 1) * half_size + (size_t)head * N * P;
+    float* __restrict__ after = slot + batch.state_offset + (size_t)(p & 1) * half_size + (size_t)head * N * P;
+    const int columns = P / VEC;                       // threads of a row of S
+    const int lanes = min(columns, LS_THREADS), per_pass = LS_THREADS / lanes;
+    const int r0 = threadIdx.x / lanes, c0 = threadIdx.x - r0 * lanes;
+    for (int cb = 0; cb < columns; cb += lanes) {      // (more than one pass only where a row has more columns than threads)
+        const int c = cb + c0;
+        float acc[VEC];
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) acc[e] = 0.0f;
+        if (r0 < per_pass && c < columns) {
+            float ve[VEC];
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) ve[e] = v[c * VEC + e];
+            constexpr int AHEAD = 8;
+            for (int n0 = r0; n0 < N; n0 += per_pass * AHEAD) {
+                float old[AHEAD][VEC];
+#pragma unroll
+                for (int u = 0; u < AHEAD; ++u) {
+                    const int n = n0 + u * per_pass;
+                    if (VEC == 4) {
+                        const float4 x = p > 0 && n < N ? *(const float4*)(before + (size_t)n * P + c * 4) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+                        old[u][0] = x.x; old[u][1 % VEC] = x.y; old[u][2 % VEC] = x.z; old[u][3 % VEC] = x.w;
+                    } else {
+                        old[u][0] = p > 0 && n < N ? before[(size_t)n * P + c] : 0.0f;
+                    }
+                }
+#pragma unroll
+                for (int u = 0; u < AHEAD; ++u) {
+                    const int n = n0 + u * per_pass;
+                    if (n >= N) break;
+                    float fresh[VEC];
+#pragma unroll
+                    for (int e = 0; e < VEC; ++e) {
+                        fresh[e] = fmaf(a, old[u][e], k[n] * ve[e]);
+                        acc[e] = fmaf(fresh[e], q[n], acc[e]);
+                    }
+                    if (VEC == 4) *(float4*)(after + (size_t)n * P + c * 4) = make_float4(fresh[0], fresh[1 % VEC], fresh[2 % VEC], fresh[3 % VEC]);
+                    else after[(size_t)n * P + c] = fresh[0];
+                }
+            }
+        }
+        __syncthreads();
+#pragma unroll
+        for (int e = 0; e < VEC; ++e)
+            if (r0 < per_pass) partial[(r0 * lanes + c0) * VEC + e] = acc[e];
+        __syncthreads();
+        for (int i = threadIdx.x; i < lanes * VEC; i += LS_THREADS) {
+            const int e = cb * VEC + i;
+            if (e >= P) continue;
+            float o = head_numbers[1] * v[e];
+            for (int r = 0; r < per_pass; ++r) o += partial[r * lanes * VEC + i];
+            out[((size_t)t * H + head) * P + e] = o;
+        }
+    }
+}
+
+// ---- longer steps ----------------------------------------------------------------------------------------------
+// l[j], c[j] and the sums of l behind every token of a chunk, in shared memory.  Called by the whole block.
+template <int CH>
+__device__ __forceinline__ void chunk_exponents(float* l, float* c, const LinearStateDecay& decay, int H, int head, int first,
+                                                int L) {
+    const float constant = decay.decay ? ls_log(decay.decay[head]) : 0.0f;
+    for (int j = threadIdx.x; j < CH; j += LS_THREADS) {
+        l[j] = j < L ? (decay.decay ? constant : decay.log_decay[(size_t)(first + j) * H + head]) : 0.0f;
+        c[j] = j < L ? (decay.key_scale ? decay.key_scale[(size_t)(first + j) * H + head] : 1.0f) : 0.0f;
+    }
+}
+
+// exp of the sum of l over the tokens from .. to of a chunk (one product where the decay is one number per head)
+__device__ __forceinline__ float span_decay(const float* l, int from, int to, bool constant) {
+    if (to < from) return 1.0f;
+    if (constant) return expf((float)(to - from + 1) * l[0]);
+    float sum = 0.0f;
+    for (int i = from; i <= to; ++i) sum += l[i];
+    return expf(sum);
+}
+
+// sums [seqs][max_chunks][heads][dim][vdim], factors [seqs][max_chunks][heads].  Threads in 16 x 16, each with RN rows and
+// four columns of S; a tile of 16 RN x 64 at a time.
+template <int CH, int RN>
+__global__ void __launch_bounds__(LS_THREADS)
+linear_state_sum_kernel(const float* __restrict__ rows, float* __restrict__ sums, float* __restrict__ factors, int max_chunks,
+                        const LinearStateShape shape, const LinearStateDecay decay, const int* __restrict__ cu_q) {
+    extern __shared__ __align__(16) float ls_smem[];
+    constexpr int TN = 16 * RN;
+    const int H = shape.heads, N = shape.dim, P = shape.vdim;
+    float* ks = ls_smem;                                  // [CH][TN], weighed
+    float* vs = ks + CH * TN;                             // [CH][64]
+    float* l = vs + CH * 64;                              // [CH]
+    float* c = l + CH;                                    // [CH]
+    float* w = c + CH;                                    // [CH]
+    pdl_launch_dependents();
+    pdl_wait();
+    const int chunk = blockIdx.x, head = blockIdx.y, s = blockIdx.z, g = head / (H / shape.groups);
+    const int first = cu_q[s] + chunk * CH, L = min(CH, cu_q[s + 1] - first);
+    if (L <= 0) return;
+    chunk_exponents<CH>(l, c, decay, H, head, first, L);
+    __syncthreads();
+    const bool constant = decay.decay != nullptr;
+    for (int j = threadIdx.x; j < L; j += LS_THREADS) w[j] = c[j] * span_decay(l, j + 1, L - 1, constant);
+    const size_t place = ((size_t)s * max_chunks + chunk) * H + head;
+    if (threadIdx.x == LS_THREADS - 1) factors[place] = span_decay(l, 0, L - 1, constant);
+    __syncthreads();
+    float* mine = sums + place * (size_t)N * P;
+    const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+    const bool vec = ((shape.row_stride | shape.k_at | shape.v_at | N | P) & 3) == 0;
+    for (int n0 = 0; n0 < N; n0 += TN) {
+        if (vec) {
+            for (int idx = threadIdx.x; idx < L * (TN / 4); idx += LS_THREADS) {
+                const int j = idx / (TN / 4), n = (idx - j * (TN / 4)) * 4;
+                float4 x = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+                if (n0 + n < N) {
+                    x = *(const float4*)(rows + (size_t)(first + j) * shape.row_stride + shape.k_at + g * N + n0 + n);
+                    if (shape.silu) x = make_float4(ls_silu(x.x), ls_silu(x.y), ls_silu(x.z), ls_silu(x.w));
+                }
+                const float wj = w[j];
+                *(float4*)(ks + j * TN + n) = make_float4(x.x * wj, x.y * wj, x.z * wj, x.w * wj);
+            }
+        } else {
+            for (int idx = threadIdx.x; idx < L * TN; idx += LS_THREADS) {
+                const int j = idx / TN, n = idx - j * TN;
+                ks[idx] = n0 + n < N ? ls_read(rows + (size_t)(first + j) * shape.row_stride + shape.k_at + g * N + n0 + n, shape.silu) * w[j] : 0.0f;
+            }
+        }
+        for (int e0 = 0; e0 < P; e0 += 64) {
+            if (n0 == 0 || P > 64) {                      // (one tile of values stays for all tiles of keys)
+                if (vec) {
+                    for (int idx = threadIdx.x; idx < L * 16; idx += LS_THREADS) {
+                        const int j = idx >> 4, e = (idx & 15) * 4;
+                        float4 x = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+                        if (e0 + e < P) {
+                            x = *(const float4*)(rows + (size_t)(first + j) * shape.row_stride + shape.v_at + head * P + e0 + e);
+                            if (shape.silu) x = make_float4(ls_silu(x.x), ls_silu(x.y), ls_silu(x.z), ls_silu(x.w));
+                        }
+                        *(float4*)(vs + j * 64 + e) = x;
+                    }
+                } else {
+                    for (int idx = threadIdx.x; idx < L * 64; idx += LS_THREADS) {
+                        const int j = idx >> 6, e = idx & 63;
+                        vs[idx] = e0 + e < P ? ls_read(rows + (size_t)(first + j) * shape.row_stride + shape.v_at + head * P + e0 + e, shape.silu) : 0.0f;
+                    }
+                }
+            }
+            __syncthreads();
+            float acc[RN][4];
+#pragma unroll
+            for (int i = 0; i < RN; ++i)
+#pragma unroll
+                for (int jj = 0; jj < 4; ++jj) acc[i][jj] = 0.0f;
+#pragma unroll 4
+            for (int j = 0; j < L; ++j) {
+                float kr[RN];
+#pragma unroll
+                for (int i = 0; i < RN; i += 4) {
+                    const float4 x = *(const float4*)(ks + j * TN + (i / 4) * 64 + ty * 4);
+                    kr[i] = x.x; kr[i + 1] = x.y; kr[i + 2] = x.z; kr[i + 3] = x.w;
+                }
+                const float4 ve = *(const float4*)(vs + j * 64 + tx * 4);
+#pragma unroll
+                for (int i = 0; i < RN; ++i) {
+                    acc[i][0] = fmaf(kr[i], ve.x, acc[i][0]); acc[i][1] = fmaf(kr[i], ve.y, acc[i][1]);
+                    acc[i][2] = fmaf(kr[i], ve.z, acc[i][2]); acc[i][3] = fmaf(kr[i], ve.w, acc[i][3]);
+                }
+            }
+#pragma unroll
+            for (int i = 0; i < RN; ++i) {
+                const int n = n0 + (i / 4) * 64 + ty * 4 + (i & 3), e = e0 + tx * 4;
+                if (n >= N || e >= P) continue;
+                float* to = mine + (size_t)n * P + e;
+                if (vec) {
+                    *(float4*)to = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
+                } else {
+#pragma unroll
+                    for (int jj = 0; jj < 4; ++jj)
+                        if (e + jj < P) to[jj] = acc[i][jj];
+                }
+            }
+            __syncthreads();
+        }
+    }
+}
+
+// Walks a sequence's chunks: every chunk's sum is replaced by the state before the chunk; the state after the last chunk
+// goes to the cache.  Several chunks' sums are fetched before any state is stored over them (a store between two loads of
+// the same array would make each load wait for the one before).
+__global__ void __launch_bounds__(LS_THREADS)
+linear_state_carry_kernel(float* __restrict__ sums, const float* __restrict__ factors, int max_chunks, int chunk_len,
+                          const LinearStateShape shape, const LinearStateBatch batch) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int H = shape.heads, cells = shape.dim * shape.vdim;
+    const int head = blockIdx.y, s = blockIdx.z;
+    const int at = blockIdx.x * LS_THREADS + threadIdx.x;
+    if (at >= cells) return;
+    const int first = batch.cu_q[s], count = batch.cu_q[s + 1] - first;
+    if (count <= 0) return;
+    const int p_first = batch.positions[first], p_last = p_first + count - 1;
+    const size_t half_size = (size_t)H * cells, mine = (size_t)head * cells + at;
+    float* slot = batch.state + (size_t)batch.slot_ids[s] * batch.state_stride + batch.state_offset;
+    float S = p_first > 0 ? slot[(size_t)((p_first - 1) & 1) * half_size + mine] : 0.0f;
+    const int chunks = (count + chunk_len - 1) / chunk_len;
+    float* cell = sums + (size_t)s * max_chunks * half_size + mine;
+    const float* factor = factors + (size_t)s * max_chunks * H + head;
+    constexpr int AHEAD = 8;
+    for (int c0 = 0; c0 < chunks; c0 += AHEAD) {
+        float own[AHEAD], f[AHEAD];
+#pragma unroll
+        for (int i = 0; i < AHEAD; ++i) {
+            own[i] = c0 + i < chunks ? __ldcg(cell + (size_t)(c0 + i) * half_size) : 0.0f;
+            f[i] = c0 + i < chunks ? __ldcg(factor + (size_t)(c0 + i) * H) : 0.0f;
+        }
+#pragma unroll
+        for (int i = 0; i < AHEAD; ++i)
+            if (c0 + i < chunks) {
+                cell[(size_t)(c0 + i) * half_size] = S;
+                S = fmaf(f[i], S, own[i]);
+            }
+    }
+    slot[(size_t)(p_last & 1) * half_size + mine] = S;
+}
+
+// Rows of a chunk, transposed into shared memory: to[n][i] (rows LD apart) = x of token i, number n; zero beyond N and L.
+template <int CH, int LD>
+__device__ __forceinline__ void load_transposed(float* to, const float* __restrict__ from, int row_stride, int N, int n_pad,
+                                                int L, int silu, bool vec) {
+    if (vec) {
+        // eight tokens by four 16-byte pieces a warp: whole sectors of every row, and two-way bank conflicts at most
+        const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+        const int pieces = n_pad >> 2;
+        constexpr int ROWS = CH / 8;
+        const int rounds = ROWS * ((pieces + 3) >> 2);
+        for (int r = warp; r < rounds; r += LS_THREADS / 32) {
+            const int i = (r % ROWS) * 8 + (lane & 7), piece = (r / ROWS) * 4 + (lane >> 3);
+            if (piece >= pieces) continue;
+            float4 x = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            if (i < L && piece * 4 < N) {
+                x = *(const float4*)(from + (size_t)i * row_stride + piece * 4);
+                if (silu) x = make_float4(ls_silu(x.x), ls_silu(x.y), ls_silu(x.z), ls_silu(x.w));
+            }
+            float* at = to + piece * 4 * LD + i;
+            at[0] = x.x; at[LD] = x.y; at[2 * LD] = x.z; at[3 * LD] = x.w;
+        }
+        return;
+    }
+    for (int idx = threadIdx.x; idx < CH * n_pad; idx += LS_THREADS) {
+        const int i = idx / n_pad, n = idx - i * n_pad;
+        to[n * LD + i] = i < L && n < N ? ls_read(from + (size_t)i * row_stride + n, silu) : 0.0f;
+    }
+}
+
+// The outputs of one chunk of one head; sums holds the state before every chunk (what linear_state_carry_kernel left).
+// Threads in 16 x 16, each with CH / 16 tokens and four columns.  n_pad: dim rounded up to a multiple of 4.
+template <int CH>
+__global__ void __launch_bounds__(LS_THREADS)
+linear_state_output_kernel(const float* __restrict__ rows, const float* __restrict__ sums, float* __restrict__ out,
+                           int max_chunks, int n_pad, const LinearStateShape shape, const LinearStateDecay decay,
+                           const int* __restrict__ cu_q) {
+    extern __shared__ __align__(16) float ls_smem[];
+    constexpr int LD = CH + 4, RI = CH / 16;              // a thread's tokens, and its keys in the scores
+    const int H = shape.heads, N = shape.dim, P = shape.vdim;
+    float* qT = ls_smem;                                  // [n_pad][LD]
+    float* kT = qT + n_pad * LD;                          // [n_pad][LD]; then the state's tile [n_pad][64]
+    float* wT = kT + n_pad * (LD > 64 ? LD : 64);         // [CH][LD]: the scores, indexed [key][query]
+    float* vs = wT + CH * LD;                             // [CH][64]
+    float* l = vs + CH * 64;                              // [CH]
+    float* c = l + CH;                                    // [CH]
+    pdl_launch_dependents();
+    pdl_wait();
+    const int chunk = blockIdx.x, head = blockIdx.y, s = blockIdx.z, g = head / (H / shape.groups);
+    const int first = cu_q[s] + chunk * CH, L = min(CH, cu_q[s + 1] - first);
+    if (L <= 0) return;
+    const bool vec_qk = ((shape.row_stride | shape.q_at | shape.k_at | N) & 3) == 0;
+    const bool vec_v = ((shape.row_stride | shape.v_at | P) & 3) == 0;
+    const float* base = rows + (size_t)first * shape.row_stride;
+    chunk_exponents<CH>(l, c, decay, H, head, first, L);
+    load_transposed<CH, LD>(qT, base + shape.q_at + g * N, shape.row_stride, N, n_pad, L, shape.silu, vec_qk);
+    load_transposed<CH, LD>(kT, base + shape.k_at + g * N, shape.row_stride, N, n_pad, L, shape.silu, vec_qk);
+    __syncthreads();
+    const bool constant = decay.decay != nullptr;
+    const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+    const int i0 = ty * RI, j0 = tx * RI;
+    {
+        float acc[RI][RI];
+#pragma unroll
+        for (int a = 0; a < RI; ++a)
+#pragma unroll
+            for (int b = 0; b < RI; ++b) acc[a][b] = 0.0f;
+        if (j0 <= i0) {
+#pragma unroll 4
+            for (int n = 0; n < n_pad; ++n) {
+                float qi[RI], kj[RI];
+                if (RI == 4) {
+                    const float4 a = *(const float4*)(qT + n * LD + i0), b = *(const float4*)(kT + n * LD + j0);
+                    qi[0] = a.x; qi[1 % RI] = a.y; qi[2 % RI] = a.z; qi[3 % RI] = a.w;
+                    kj[0] = b.x; kj[1 % RI] = b.y; kj[2 % RI] = b.z; kj[3 % RI] = b.w;
+                } else {
+#pragma unroll
+                    for (int a = 0; a < RI; ++a) { qi[a] = qT[n * LD + i0 + a]; kj[a] = kT[n * LD + j0 + a]; }
+                }
+#pragma unroll
+                for (int a = 0; a < RI; ++a)
+#pragma unroll
+                    for (int b = 0; b < RI; ++b) acc[a][b] = fmaf(qi[a], kj[b], acc[a][b]);
+            }
+        }
+        // the exponents between: what lies between the two tiles, then the tokens inside either
+        float between = 0.0f;
+        if (!constant && j0 < i0)
+            for (int i = j0 + RI; i <= i0; ++i) between += l[i];
+#pragma unroll
+        for (int b = 0; b < RI; ++b) {
+            const int j = j0 + b;
+            float sum = between;
+            if (j0 < i0) {
+#pragma unroll
+                for (int x = RI - 1; x > 0; --x)
+                    if (x > b) sum += l[j0 + x];
+            }
+#pragma unroll
+            for (int a = 0; a < RI; ++a) {
+                const int i = i0 + a;
+                float weight = 0.0f;
+                if (j <= i && i < L) {
+                    float exponent;
+                    if (constant) {
+                        exponent = i == j ? 0.0f : (float)(i - j) * l[0];
+                    } else if (j0 < i0) {
+                        if (a > 0) sum += l[i];
+                        exponent = sum;
+                    } else {
+                        exponent = 0.0f;
+                        for (int x = j + 1; x <= i; ++x) exponent += l[x];
+                    }
+                    weight = acc[a][b] * expf(exponent) * c[j];
+                }
+                wT[j * LD + i] = weight;
+            }
+        }
+    }
+    float carry[RI];
+#pragma unroll
+    for (int a = 0; a < RI; ++a) carry[a] = i0 + a < L ? span_decay(l, 0, i0 + a, constant) : 0.0f;
+    const float skip = decay.skip ? decay.skip[head] : 0.0f;
+    const float* before = sums + (((size_t)s * max_chunks + chunk) * H + head) * (size_t)N * P;
+    float* st = kT;
+    const int j_end = min(L, (i0 / RI | 1) * RI + RI);    // (the two rows of threads of a warp walk the same keys)
+    for (int e0 = 0; e0 < P; e0 += 64) {
+        __syncthreads();                                  // the scores are in place; the tiles before have been read
+        if (vec_v) {
+            for (int idx = threadIdx.x; idx < CH * 16; idx += LS_THREADS) {
+                const int j = idx >> 4, e = (idx & 15) * 4;
+                float4 x = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+                if (j < L && e0 + e < P) {
+                    x = *(const float4*)(base + (size_t)j * shape.row_stride + shape.v_at + head * P + e0 + e);
+                    if (shape.silu) x = make_float4(ls_silu(x.x), ls_silu(x.y), ls_silu(x.z), ls_silu(x.w));
+                }
+                *(float4*)(vs + j * 64 + e) = x;
+            }
+            for (int idx = threadIdx.x; idx < N * 16; idx += LS_THREADS) {
+                const int n = idx >> 4, e = (idx & 15) * 4;
+                *(float4*)(st + n * 64 + e) = e0 + e < P ? *(const float4*)(before + (size_t)n * P + e0 + e) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            }
+        } else {
+            for (int idx = threadIdx.x; idx < CH * 64; idx += LS_THREADS) {
+                const int j = idx >> 6, e = idx & 63;
+                vs[idx] = j < L && e0 + e < P ? ls_read(base + (size_t)j * shape.row_stride + shape.v_at + head * P + e0 + e, shape.silu) : 0.0f;
+            }
+            for (int idx = threadIdx.x; idx < N * 64; idx += LS_THREADS) {
+                const int n = idx >> 6, e = idx & 63;
+                st[idx] = e0 + e < P ? before[(size_t)n * P + e0 + e] : 0.0f;
+            }
+        }
+        __syncthreads();
+        float acc[RI][4];
+#pragma unroll
+        for (int a = 0; a < RI; ++a)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) acc[a][e] = 0.0f;
+#pragma unroll 4
+        for (int n = 0; n < N; ++n) {                     // what the state before the chunk gives
+            const float4 sv = *(const float4*)(st + n * 64 + tx * 4);
+            float qi[RI];
+            if (RI == 4) {
+                const float4 a = *(const float4*)(qT + n * LD + i0);
+                qi[0] = a.x; qi[1 % RI] = a.y; qi[2 % RI] = a.z; qi[3 % RI] = a.w;
+            } else {
+#pragma unroll
+                for (int a = 0; a < RI; ++a) qi[a] = qT[n * LD + i0 + a];
+            }
+#pragma unroll
+            for (int a = 0; a < RI; ++a) {
+                acc[a][0] = fmaf(qi[a], sv.x, acc[a][0]); acc[a][1] = fmaf(qi[a], sv.y, acc[a][1]);
+                acc[a][2] = fmaf(qi[a], sv.z, acc[a][2]); acc[a][3] = fmaf(qi[a], sv.w, acc[a][3]);
+            }
+        }
+#pragma unroll
+        for (int a = 0; a < RI; ++a)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) acc[a][e] *= carry[a];
+#pragma unroll 4
+        for (int j = 0; j < j_end; ++j) {                 // what the chunk's own tokens give
+            const float4 ve = *(const float4*)(vs + j * 64 + tx * 4);
+            float wi[RI];
+            if (RI == 4) {
+                const float4 a = *(const float4*)(wT + j * LD + i0);
+                wi[0] = a.x; wi[1 % RI] = a.y; wi[2 % RI] = a.z; wi[3 % RI] = a.w;
+            } else {
+#pragma unroll
+                for (int a = 0; a < RI; ++a) wi[a] = wT[j * LD + i0 + a];
+            }
+#pragma unroll
+            for (int a = 0; a < RI; ++a) {
+                acc[a][0] = fmaf(wi[a], ve.x, acc[a][0]); acc[a][1] = fmaf(wi[a], ve.y, acc[a][1]);
+                acc[a][2] = fmaf(wi[a], ve.z, acc[a][2]); acc[a][3] = fmaf(wi[a], ve.w, acc[a][3]);
+            }
+        }
+        const int e = e0 + tx * 4;
+#pragma unroll
+        for (int a = 0; a < RI; ++a) {
+            const int i = i0 + a;
+            if (i >= L || e >= P) continue;
+            const float4 own = *(const float4*)(vs + i * 64 + tx * 4);
+            const float o[4] = {fmaf(skip, own.x, acc[a][0]), fmaf(skip, own.y, acc[a][1]), fmaf(skip, own.z, acc[a][2]),
+                                fmaf(skip, own.w, acc[a][3])};
+            float* to = out + ((size_t)(first + i) * H + head) * P + e;
+            if ((P & 3) == 0) {
+                *(float4*)to = make_float4(o[0], o[1], o[2], o[3]);
+            } else {
+#pragma unroll
+                for (int x = 0; x < 4; ++x)
+                    if (e + x < P) to[x] = o[x];
+            }
+        }
+    }
+}
+
+// ---- Mamba-2's steps between its input projection and the recurrence, for steps of more than one token a sequence --------
+// A thread takes one channel of CONV_TOKENS neighbouring tokens and keeps the last inputs in registers (up to 8 taps).
+constexpr int CONV_TOKENS = 16, CONV_HELD = 8;
+
+__global__ void __launch_bounds__(256)
+conv_silu_kernel(const float* __restrict__ rows, int row_stride, const float* __restrict__ conv_w,
+                 const float* __restrict__ conv_b, int channels, int taps, float* __restrict__ out, int n_tokens,
+                 const int* __restrict__ positions, const int* __restrict__ token_seq, const int* __restrict__ cu_q,
+                 const int* __restrict__ slot_ids, const float* __restrict__ state, long long state_stride,
+                 long long ring_offset) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int c = blockIdx.x * blockDim.x + threadIdx.x;
+    if (c >= channels) return;
+    const int t0 = blockIdx.y * CONV_TOKENS, t1 = min(n_tokens, t0 + CONV_TOKENS);
+    const float bias = conv_b[c];
+    const float* weights = conv_w + (size_t)c * taps;
+    const bool held = taps <= CONV_HELD;
+    float w[CONV_HELD], u[CONV_HELD];                     // w[b], u[b]: the weight and the input of the token b back
+#pragma unroll
+    for (int b = 0; b < CONV_HELD; ++b) { w[b] = held && b < taps ? weights[taps - 1 - b] : 0.0f; u[b] = 0.0f; }
+    int seq = -1;
+    for (int t = t0; t < t1; ++t) {
+        const int s = token_seq[t], p = positions[t];
+        float sum = bias;
+        if (held) {
+            if (s != seq) {                               // this block's first token of a sequence: fetch what lies before it
+                seq = s;
+                const int first = cu_q[s];
+                const float* ring = state + (size_t)slot_ids[s] * state_stride + ring_offset;
+#pragma unroll
+                for (int b = 1; b < CONV_HELD; ++b) {
+                    float x = 0.0f;
+                    if (b < taps && p - b >= 0)
+                        x = t - b >= first ? rows[(size_t)(t - b) * row_stride + c] : ring[(size_t)((p - b) % taps) * channels + c];
+                    u[b] = x;
+                }
+            }
+            u[0] = rows[(size_t)t * row_stride + c];
+#pragma unroll
+            for (int b = CONV_HELD - 1; b >= 0; --b) sum = fmaf(w[b], u[b], sum);
+#pragma unroll
+            for (int b = CONV_HELD - 1; b > 0; --b) u[b] = u[b - 1];
+        } else {
+            const int first = cu_q[s];
+            const float* ring = state + (size_t)slot_ids[s] * state_stride + ring_offset;
+            for (int j = 0; j < taps; ++j) {
+                const int back = taps - 1 - j;
+                if (p - back < 0) continue;
+                const float x = t - back >= first ? rows[(size_t)(t - back) * row_stride + c] : ring[(size_t)((p - back) % taps) * channels + c];
+                sum = fmaf(weights[j], x, sum);
+            }
+        }
+        out[(size_t)t * channels + c] = ls_silu(sum);
+    }
+}
+
+// dt[t][h] = softplus(row's step size + dt_bias[h]), log_decay[t][h] = -exp(a_log[h]) dt[t][h].
+__global__ void __launch_bounds__(256)
+step_sizes_kernel(const float* __restrict__ rows, int row_stride, int dt_at, const float* __restrict__ dt_bias,
+                  const float* __restrict__ a_log, int heads, int n_tokens, float* __restrict__ dt, float* __restrict__ log_decay) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const long long item = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (item >= (long long)n_tokens * heads) return;
+    const int t = (int)(item / heads), h = (int)(item - (long long)t * heads);
+    const float step = ls_softplus(rows[(size_t)t * row_stride + dt_at + h] + dt_bias[h]);
+    dt[item] = step;
+    log_decay[item] = -expf(a_log[h]) * step;
+}
+
+// ---- a norm with a gate ------------------------------------------------------------------------------------------------
+// out = gated norm of float rows y [tokens, width]: the row in `groups` equal parts, each divided by its own root mean
+// square, times a weight, and a gate on every number: gate_first, silu(gate) before the norm; else sigmoid(gate) after it.
+// A block per (token, part); the part stays in shared memory between the two passes.
+template <typename T>
+__global__ void __launch_bounds__(256)
+gated_norm_kernel(const float* __restrict__ y, const float* __restrict__ gate, int gate_stride, const float* __restrict__ weight,
+                  int width, int groups, float eps, int gate_first, T* __restrict__ out, int out_stride) {
+    extern __shared__ __align__(16) float gn_part[];
+    __shared__ float scratch[33];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t = blockIdx.x, part = blockIdx.y, size = width / groups, at = part * size;
+    const float* row = y + (size_t)t * width + at;
+    const float* g = gate + (size_t)t * gate_stride + at;
+    T* to = out + (size_t)t * out_stride + at;
+    const float* w = weight + at;
+    float squares = 0.0f;
+    const bool vec = ((size | width | gate_stride | out_stride) & 3) == 0 &&
+                     (((uintptr_t)y | (uintptr_t)gate | (uintptr_t)weight | (uintptr_t)out) & 15) == 0;
+    if (vec) {
+        for (int i = 4 * threadIdx.x; i < size; i += 1024) {
+            float4 v = *(const float4*)(row + i);
+            if (gate_first) {
+                const float4 z = *(const float4*)(g + i);
+                v.x *= ls_silu(z.x); v.y *= ls_silu(z.y); v.z *= ls_silu(z.z); v.w *= ls_silu(z.w);
+            }
+            squares = fmaf(v.x, v.x, squares); squares = fmaf(v.y, v.y, squares);
+            squares = fmaf(v.z, v.z, squares); squares = fmaf(v.w, v.w, squares);
+            *(float4*)(gn_part + i) = v;
+        }
+    } else {
+        for (int i = threadIdx.x; i < size; i += 256) {
+            float v = row[i];
+            if (gate_first) v *= ls_silu(g[i]);
+            squares = fmaf(v, v, squares);
+            gn_part[i] = v;
+        }
+    }
+    const float factor = 1.0f / sqrtf(block_sum(squares, scratch) / (float)size + eps);
+    if (vec) {
+        for (int i = 4 * threadIdx.x; i < size; i += 1024) {
+            float4 v = *(const float4*)(gn_part + i);
+            const float4 x = *(const float4*)(w + i);
+            v.x *= factor * x.x; v.y *= factor * x.y; v.z *= factor * x.z; v.w *= factor * x.w;
+            if (!gate_first) {
+                const float4 z = *(const float4*)(g + i);
+                v.x /= 1.0f + expf(-z.x); v.y /= 1.0f + expf(-z.y); v.z /= 1.0f + expf(-z.z); v.w /= 1.0f + expf(-z.w);
+            }
+            if (sizeof(T) == 4) {
+                *(float4*)(to + i) = v;
+            } else {
+                const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+                *(uint2*)(to + i) = make_uint2(*(const uint32_t*)&lo, *(const uint32_t*)&hi);
+            }
+        }
+    } else {
+        for (int i = threadIdx.x; i < size; i += 256) {
+            float v = gn_part[i] * factor * w[i];
+            if (!gate_first) v /= 1.0f + expf(-g[i]);
+            to[i] = from_float<T>(v);
+        }
+    }
+    if (part == groups - 1)
+        for (int i = width + threadIdx.x; i < out_stride; i += 256) out[(size_t)t * out_stride + i] = from_float<T>(0.0f);
+}
+
+static int ls_reserve(const void* kernel, size_t bytes, const char* name) {
+    if (bytes <= 48 * 1024) return 0;
+    if (bytes > 220 * 1024) return fail(name, "the sizes are too large for this kernel's shared memory");
+    if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes) != cudaSuccess)
+        return fail(name, "cannot reserve shared memory");
+    return 0;
+}
+
+static size_t ls_output_smem(int ch, int dim) {
+    const int n_pad = (dim + 3) & ~3, ld = ch + 4;
+    return (size_t)(n_pad * ld + n_pad * (ld > 64 ? ld : 64) + ch * ld + ch * 64 + 2 * ch) * sizeof(float);
+}
+
+// The longest chunk whose tiles fit: 64 tokens, 32, or 16.
+static int ls_chunk(int dim) {
+    return ls_output_smem(64, dim) <= 200 * 1024 ? 64 : (ls_output_smem(32, dim) <= 200 * 1024 ? 32 : 16);
+}
+
+static int ls_check(const char* name, const LinearStateShape& shape, const LinearStateBatch& batch) {
+    if (shape.heads <= 0 || shape.groups <= 0 || shape.heads % shape.groups || shape.dim <= 0 || shape.vdim <= 0)
+        return fail(name, "heads must be a positive multiple of the query and key heads, and sizes positive");
+    if (shape.heads > 65535) return fail(name, "too many heads");
+    const int qk = shape.groups * shape.dim, v = shape.heads * shape.vdim;
+    if (shape.q_at < 0 || shape.k_at < 0 || shape.v_at < 0 || shape.q_at + qk > shape.row_stride ||
+        shape.k_at + qk > shape.row_stride || shape.v_at + v > shape.row_stride)
+        return fail(name, "queries, keys and values must lie inside a row");
+    if (!batch.positions || !batch.cu_q || !batch.slot_ids || !batch.state)
+        return fail(name, "the step's metadata and the state are needed");
+    if (batch.state_offset < 0 || batch.state_offset + 2LL * shape.heads * shape.dim * shape.vdim > batch.state_stride)
+        return fail(name, "a slot's state is too small: 2 * heads * dim * vdim floats are needed");
+    return 0;
+}
+
+}  // namespace skv
+
+using namespace skv;
+
+// Floats of scratch for a step whose longest sequence brings max_q_len tokens (0 for one token a sequence).
+SKV_EXPORT long long skv_linear_state_scratch(int n_seqs, int max_q_len, int heads, int dim, int vdim) {
+    if (max_q_len <= 1) return 0;
+    const int ch = ls_chunk(dim);
+    return (long long)n_seqs * ((max_q_len + ch - 1) / ch) * heads * ((long long)dim * vdim + 1);
+}
+
+// rows: float [n_tokens, row_stride]; out: float [n_tokens, heads * vdim].  decay [heads], or log_decay [n_tokens, heads];
+// key_scale [n_tokens, heads] and skip [heads] may be null.  state: float [slots][state_stride].
+SKV_EXPORT int skv_linear_state(const float* rows, int row_stride, int q_at, int k_at, int v_at, int silu, const float* decay,
+                                const float* log_decay, const float* key_scale, const float* skip, float* out,
+                                float* scratch, int n_tokens, int n_seqs, int heads, int groups, int dim, int vdim,
+                                int max_q_len, const int* positions, const int* token_seq, const int* cu_q,
+                                const int* slot_ids, float* state, long long state_stride, long long state_offset,
+                                cudaStream_t stream) {
+    const char* name = "skv_linear_state";
+    if (n_tokens <= 0 || n_seqs <= 0) return 0;
+    if (!rows || !out || (!decay && !log_decay)) return fail(name, "rows, a decay and a place for the result are needed");
+    if (n_seqs > 65535 || max_q_len <= 0) return fail(name, "too many sequences in one step, or no tokens");
+    const LinearStateShape shape = {heads, groups, dim, vdim, row_stride, q_at, k_at, v_at, silu};
+    const LinearStateDecay decays = {decay, log_decay, key_scale, skip};
+    const LinearStateBatch batch = {positions, cu_q, slot_ids, state, state_stride, state_offset};
+    if (int code = ls_check(name, shape, batch)) return code;
+    if (((uintptr_t)rows | (uintptr_t)out | (uintptr_t)state | (uintptr_t)scratch) & 15) return fail(name, "operands must be 16-byte aligned");
+    if (max_q_len == 1) {
+        if (n_tokens != n_seqs) return fail(name, "one token a sequence means as many tokens as sequences");
+        ConvStep none = {};
+        const bool vec = vdim % 4 == 0 && state_stride % 4 == 0 && state_offset % 4 == 0;
+        const size_t smem = (size_t)(2 * ((dim + 3) & ~3) + ((vdim + 3) & ~3) + LS_THREADS * (vec ? 4 : 1)) * sizeof(float);
+        auto kernel = vec ? linear_state_step_kernel<4> : linear_state_step_kernel<1>;
+        if (int code = ls_reserve((const void*)kernel, smem, name)) return code;
+        return launch_pdl(name, kernel, dim3(heads, n_seqs), dim3(LS_THREADS), smem, stream, rows, out, shape, decays, none, batch);
+    }
+    if (!scratch) return fail(name, "a step of more than one token a sequence needs scratch for its chunks");
+    const int ch = ls_chunk(dim), max_chunks = (max_q_len + ch - 1) / ch;
+    if (ls_output_smem(ch, dim) > 220 * 1024) return fail(name, "the head size is too large for this kernel's shared memory");
+    float* sums = scratch;
+    float* factors = scratch + (size_t)n_seqs * max_chunks * heads * dim * vdim;
+    const bool wide = dim > 64;
+    const dim3 grid(max_chunks, heads, n_seqs);
+    {
+        const size_t smem = (size_t)(ch * (wide ? 128 : 64) + ch * 64 + 3 * ch) * sizeof(float);
+        auto kernel = ch == 64 ? (wide ? linear_state_sum_kernel<64, 8> : linear_state_sum_kernel<64, 4>)
+                     : ch == 32 ? (wide ? linear_state_sum_kernel<32, 8> : linear_state_sum_kernel<32, 4>)
+                                : (wide ? linear_state_sum_kernel<16, 8> : linear_state_sum_kernel<16, 4>);
+        if (int code = ls_reserve((const void*)kernel, smem, name)) return code;
+        if (int code = launch_pdl(name, kernel, grid, dim3(LS_THREADS), smem, stream, rows, sums, factors, max_chunks, shape, decays, cu_q))
+            return code;
+    }
+    if (int code = launch_pdl(name, linear_state_carry_kernel, dim3((dim * vdim + LS_THREADS - 1) / LS_THREADS, heads, n_seqs),
+                              dim3(LS_THREADS), 0, stream, sums, (const float*)factors, max_chunks, ch, shape, batch))
+        return code;
+    const size_t smem = ls_output_smem(ch, dim);
+    auto kernel = ch == 64 ? linear_state_output_kernel<64> : (ch == 32 ? linear_state_output_kernel<32> : linear_state_output_kernel<16>);
+    if (int code = ls_reserve((const void*)kernel, smem, name)) return code;
+    return launch_pdl(name, kernel, grid, dim3(LS_THREADS), smem, stream, rows, (const float*)sums, out, max_chunks,
+                      (dim + 3) & ~3, shape, decays, cu_q);
+}
+
+// One token a sequence of a Mamba-2 mixer, in one kernel: rows float [n_seqs, row_stride] hold the input projection with
+// the convolved channels first, [values: heads * vdim | keys: groups * dim | queries: groups * dim], and the step sizes at
+// dt_at.  The state of a slot holds S twice from state_offset on and the ring of the last inputs [taps][channels] from
+// ring_offset on.
+SKV_EXPORT int skv_mamba2_step(const float* rows, int row_stride, const float* conv_w, const float* conv_b, int taps, int dt_at,
+                               const float* dt_bias, const float* a_log, const float* skip, float* out, int n_seqs, int heads,
+                               int groups, int dim, int vdim, const int* positions, const int* token_seq, const int* cu_q,
+                               const int* slot_ids, float* state, long long state_stride, long long state_offset,
+                               long long ring_offset, cudaStream_t stream) {
+    const char* name = "skv_mamba2_step";
+    if (n_seqs <= 0) return 0;
+    if (!rows || !conv_w || !conv_b || !dt_bias || !a_log || !out || taps <= 0) return fail(name, "a weight or a place for the result is missing");
+    if (n_seqs > 65535) return fail(name, "too many sequences in one step");
+    const int inner = heads * vdim, channels = inner + 2 * groups * dim;
+    const LinearStateShape shape = {heads, groups, dim, vdim, row_stride, inner + groups * dim, inner, 0, 0};
+    const LinearStateDecay decays = {nullptr, nullptr, nullptr, skip};
+    const LinearStateBatch batch = {positions, cu_q, slot_ids, state, state_stride, state_offset};
+    const ConvStep conv = {conv_w, conv_b, dt_bias, a_log, taps, channels, dt_at, ring_offset};
+    if (int code = ls_check(name, shape, batch)) return code;
+    if (dt_at < 0 || dt_at + heads > row_stride || ring_offset < 0 ||
+        (taps > 1 && ring_offset + (long long)taps * channels > state_stride))
+        return fail(name, "the step sizes must lie inside a row and the ring inside a slot's state");
+    if (((uintptr_t)rows | (uintptr_t)out | (uintptr_t)state) & 15) return fail(name, "operands must be 16-byte aligned");
+    const bool vec = vdim % 4 == 0 && state_stride % 4 == 0 && state_offset % 4 == 0;
+    const size_t smem = (size_t)(2 * ((dim + 3) & ~3) + ((vdim + 3) & ~3) + LS_THREADS * (vec ? 4 : 1)) * sizeof(float);
+    auto kernel = vec ? linear_state_step_kernel<4> : linear_state_step_kernel<1>;
+    if (int code = ls_reserve((const void*)kernel, smem, name)) return code;
+    return launch_pdl(name, kernel, dim3(heads, n_seqs), dim3(LS_THREADS), smem, stream, rows, out, shape, decays, conv, batch);
+}
+
+// out [n_tokens, channels] float = silu(conv_b + causal convolution over time of the rows' first `channels` columns); what
+// lies before the step comes from the ring [taps][channels] at ring_offset of a slot's state.
+SKV_EXPORT int skv_conv_silu(const float* rows, int row_stride, const float* conv_w, const float* conv_b, int channels, int taps,
+                             float* out, int n_tokens, const int* positions, const int* token_seq, const int* cu_q,
+                             const int* slot_ids, const float* state, long long state_stride, long long ring_offset,
+                             cudaStream_t stream) {
+    if (n_tokens <= 0) return 0;
+    if (!rows || !conv_w || !conv_b || !out || !positions || !token_seq || !cu_q || !slot_ids || (taps > 1 && !state))
+        return fail("skv_conv_silu", "a pointer is missing");
+    if (channels <= 0 || taps <= 0 || row_stride < channels || (taps > 1 && (ring_offset < 0 || ring_offset + (long long)taps * channels > state_stride)))
+        return fail("skv_conv_silu", "sizes do not agree");
+    const int rows_of_blocks = (n_tokens + CONV_TOKENS - 1) / CONV_TOKENS;
+    if (rows_of_blocks > 65535) return fail("skv_conv_silu", "too many tokens in one step");
+    return launch_pdl("skv_conv_silu", conv_silu_kernel, dim3((channels + 255) / 256, rows_of_blocks), dim3(256), 0, stream, rows,
+                      row_stride, conv_w, conv_b, channels, taps, out, n_tokens, positions, token_seq, cu_q, slot_ids, state,
+                      state_stride, ring_offset);
+}
+
+SKV_EXPORT int skv_step_sizes(const float* rows, int row_stride, int dt_at, const float* dt_bias, const float* a_log, int heads,
+                              int n_tokens, float* dt, float* log_decay, cudaStream_t stream) {
+    if (n_tokens <= 0) return 0;
+    if (!rows || !dt_bias || !a_log || !dt || !log_decay || heads <= 0 || dt_at < 0 || dt_at + heads > row_stride)
+        return fail("skv_step_sizes", "the step sizes must lie inside a row");
+    const long long items = (long long)n_tokens * heads;
+    return launch_pdl("skv_step_sizes", step_sizes_kernel, dim3((unsigned)((items + 255) / 256)), dim3(256), 0, stream, rows,
+                      row_stride, dt_at, dt_bias, a_log, heads, n_tokens, dt, log_decay);
+}
+
+// y float [n, width], gate float rows gate_stride apart, weight float [width], out [n, out_stride] in the compute dtype.
+SKV_EXPORT int skv_gated_norm(const float* y, const float* gate, int gate_stride, const float* weight, int width, int groups,
+                              float eps, int gate_first, void* out, int out_stride, int n, cudaStream_t stream) {
+    if (n <= 0) return 0;
+    if (!y || !gate || !weight || !out || width <= 0 || groups <= 0 || width % groups || gate_stride < width || out_stride < width || groups > 65535)
+        return fail("skv_gated_norm", "sizes do not agree");
+    const size_t smem = (size_t)(width / groups) * sizeof(float);
+    auto kernel = gated_norm_kernel<skv_t>;
+    if (int code = ls_reserve((const void*)kernel, smem, "skv_gated_norm")) return code;
+    return launch_pdl("skv_gated_norm", kernel, dim3(n, groups), dim3(256), smem, stream, y, gate, gate_stride, weight, width,
+                      groups, eps, gate_first, (skv_t*)out, out_stride);
+}

@@ -237,7 +237,7 @@ __device__ __forceinline__ void find_tile(const int* __restrict__ offsets, int e
 template <typename TIn, typename TOut, bool GATED>
 __global__ void __launch_bounds__(256)
 expert_linear_kernel(const TIn* __restrict__ a, int a_stride, const int* __restrict__ rows, const TIn* __restrict__ w,
-                     const int* __restrict__ offsets, TOut* __restrict__ out, int experts, int N, int K, int act) {
+                     const int* __restrict__ offsets, TOut* __restrict__ out, int experts, int N, int K, act_t act_word) {
     __shared__ float as[EXP_ROWS][EXP_K + 1];
     __shared__ float ws[EXP_OUTS][EXP_K + 1];
     __shared__ float us[GATED ? EXP_OUTS : 1][EXP_K + 1];
@@ -256,6 +256,8 @@ expert_linear_kernel(const TIn* __restrict__ a, int a_stride, const int* __restr
     }
     __syncthreads();
     const int o0 = blockIdx.x * EXP_OUTS;
+    const int act = act_word < 0 ? -1 : (int)(act_word & 0xff);
+    const float limit = act_param(act_word);
     const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
     const TIn* w_e = w + (size_t)expert * (GATED ? 2 : 1) * N * K;
     float acc[2][4] = {};
@@ -304,6 +306,10 @@ expert_linear_kernel(const TIn* __restrict__ a, int a_stride, const int* __restr
             const int o = o0 + tx + 16 * j;
             if (o >= N) continue;
             float v = acc[i][j];
+            if (GATED && act == ACT_SWIGLU_CLAMP) {
+                out[(size_t)(first + r) * N + o] = from_float<TOut>(clamped_swiglu(v, up[i][j], limit));
+                continue;
+            }
             if (act == ACT_RELU2) v = relu_squared(v);
             else if (act == ACT_GELU_TANH) v = gelu_tanh(v);
             else if (act == ACT_SILU) v = v / (1.0f + expf(-v));
@@ -329,6 +335,34 @@ gather_rows_kernel(const T* __restrict__ a, int a_stride, const int* __restrict_
     for (int i = lane; i < pieces; i += 32) dst[i] = src[i];
 }
 
+// out[place[pair]] = a[token of the pair] * weights[pair] for every (token, choice) pair: the tokens' rows in sorted order
+// where the weights multiply the experts' inputs.  VEC: rows of whole 16 bytes.  A warp makes a row.
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(256)
+scatter_rows_kernel(const T* __restrict__ a, const int* __restrict__ place, const float* __restrict__ weights, int top,
+                    T* __restrict__ out, int pairs, int K) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int pair = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (pair >= pairs) return;
+    const T* src = a + (size_t)(pair / top) * K;
+    T* dst = out + (size_t)place[pair] * K;
+    const float w = weights[pair];
+    if (VEC) {
+        constexpr int EACH = 16 / (int)sizeof(T);
+        for (int i = lane; i < K / EACH; i += 32) {
+            const uint4 raw = ((const uint4*)src)[i];
+            const T* x = (const T*)&raw;
+            T y[EACH];
+#pragma unroll
+            for (int e = 0; e < EACH; ++e) y[e] = from_float<T>(to_float(x[e]) * w);
+            ((uint4*)dst)[i] = *(const uint4*)y;
+        }
+    } else {
+        for (int i = lane; i < K; i += 32) dst[i] = from_float<T>(to_float(src[i]) * w);
+    }
+}
+
 // ---- the weighted sum ----------------------------------------------------------------------------------------------
 __global__ void __launch_bounds__(256)
 combine_experts_kernel(const float* __restrict__ results, const int* __restrict__ place, const float* __restrict__ weights,
@@ -341,7 +375,7 @@ combine_experts_kernel(const float* __restrict__ results, const int* __restrict_
     const int t = blockIdx.x;
     if (threadIdx.x < top) {
         where[threadIdx.x] = place[(size_t)t * top + threadIdx.x];
-        weight[threadIdx.x] = weights[(size_t)t * top + threadIdx.x];
+        weight[threadIdx.x] = weights ? weights[(size_t)t * top + threadIdx.x] : 1.0f;
     }
     __syncthreads();
     const float gate = shared ? (share ? share[t] : 1.0f) : 0.0f;
@@ -398,24 +432,25 @@ SKV_EXPORT int skv_sort_by_expert(const int* chosen, int pairs, int top, int exp
 }
 
 // a [a_rows, a_stride] and w [experts, N, K] in the compute dtype; rows int [pairs] or null (row p reads a[p]);
-// out [pairs, N] float (out_is_float) or the compute dtype; act: an activation's code or -1 for none.
+// out [pairs, N] float (out_is_float) or the compute dtype; act: an activation's word (its code, and a parameter's bits
+// in the high half) or -1 for none.
 // gated: w is [experts, 2 N, K], tiles of 8 gate rows and their 8 up rows; out = act(gate . a) * (up . a).
 // In bfloat16, rows that lie in sorted order already (rows null, a_stride = K) with K a multiple of 8 go to the
 // tensor-memory GEMM's grouped form; `flag` is where its bounded waits report that they gave up.
 SKV_EXPORT int skv_expert_linear(const void* a, int a_stride, int a_rows, const int* rows, const void* w,
                                  const int* offsets, void* out, int out_is_float, int pairs, int experts, int N, int K,
-                                 int act, int gated, int* flag, cudaStream_t stream) {
+                                 act_t act, int gated, int* flag, cudaStream_t stream) {
     if (pairs <= 0) return 0;
     if (experts <= 0 || experts > ROUTE_MAX_EXPERTS || N <= 0 || K <= 0 || a_stride < K || a_rows <= 0)
         return fail("skv_expert_linear", "sizes do not agree");
     if (!a || !w || !offsets || !out) return fail("skv_expert_linear", "rows, weights, offsets and a place for the result are needed");
-    if (act >= ACT_SWIGLU_CLAMP) return fail("skv_expert_linear", "this activation is not served");
+    if (act >= 0 && (act & 0xff) >= (gated ? ACT_COUNT : ACT_SWIGLU_CLAMP)) return fail("skv_expert_linear", "this activation is not served");
     if (gated && (act < 0 || N % 8 != 0)) return fail("skv_expert_linear", "a gated weight needs an activation and whole tiles of 8 rows");
 #if SKV_DTYPE == SKV_BF16
     if (!rows && a_stride == K && K % 8 == 0 && a_rows >= pairs && !(((uintptr_t)a | (uintptr_t)w) & 15) &&
-        (!gated || (!out_is_float && act != ACT_RELU2)))
+        (!gated || (!out_is_float && (act & 0xff) != ACT_RELU2)))
         return grouped_linear_tcgen05(a, w, offsets, out, out_is_float, pairs, experts, gated ? 2 * N : N, K,
-                                      gated ? (act_t)act : (act >= 0 ? ((act_t)act | ACT_ON_STORE) : (act_t)0), gated,
+                                      gated ? act : (act >= 0 ? (act | ACT_ON_STORE) : (act_t)0), gated,
                                       flag, stream);
 #endif
     const int row_tiles = (pairs + EXP_ROWS - 1) / EXP_ROWS + experts;       // no expert leaves more than one part tile
@@ -446,12 +481,24 @@ SKV_EXPORT int skv_gather_rows(const void* a, int a_stride, const int* rows, voi
                       (const skv_t*)a, a_stride, rows, (skv_t*)out, pairs, K);
 }
 
+// a [pairs / top, K] and out [pairs, K] in the compute dtype: out[place[p]] = a[p / top] * weights[p].
+SKV_EXPORT int skv_scatter_rows(const void* a, const int* place, const float* weights, int top, void* out, int pairs, int K,
+                                cudaStream_t stream) {
+    if (pairs <= 0) return 0;
+    if (!a || !place || !weights || !out || K <= 0 || top <= 0) return fail("skv_scatter_rows", "rows, their places and weights are needed");
+    const bool vec = (K * sizeof(skv_t)) % 16 == 0 && (((uintptr_t)a | (uintptr_t)out) & 15) == 0;
+    auto kernel = vec ? scatter_rows_kernel<skv_t, true> : scatter_rows_kernel<skv_t, false>;
+    return launch_pdl("skv_scatter_rows", kernel, dim3((pairs + 7) / 8), dim3(256), 0, stream, (const skv_t*)a, place, weights,
+                      top, (skv_t*)out, pairs, K);
+}
+
+// weights null: every choice counts as it is.
 SKV_EXPORT int skv_combine_experts(const float* results, const int* place, const float* weights, const float* shared,
                                    const float* share, float* x, int n, int hidden, int top, int add,
                                    cudaStream_t stream) {
     if (n <= 0) return 0;
     if (hidden <= 0 || top <= 0 || top > ROUTE_MAX_TOP) return fail("skv_combine_experts", "1 to 16 choices a token are served");
-    if (!results || !place || !weights || !x || (share && !shared))
+    if (!results || !place || !x || (share && !shared))
         return fail("skv_combine_experts", "results, places, weights and the stream are needed");
     return launch_pdl("skv_combine_experts", combine_experts_kernel, dim3(n), dim3(256), 0, stream, results, place,
                       weights, shared, share, x, hidden, top, add);

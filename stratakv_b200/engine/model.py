@@ -69,7 +69,8 @@ def embedding_cache_request(spec: ModelSpec) -> Optional[CacheRequest]:
 
 def default_head_dim(spec: ModelSpec) -> int:
     for layer in spec.layers:
-        head_dim = getattr(layer.mixer, "head_dim", None)
+        # (a mixer that pads its heads names the size its kernels are built for)
+        head_dim = getattr(layer.mixer, "kernel_head_dim", None) or getattr(layer.mixer, "head_dim", None)
         if head_dim and head_dim % 16 == 0 and head_dim <= 256:      # (the sizes a library can be built for)
             return head_dim
     return 64       # no part needs a head size: any build of the library will do

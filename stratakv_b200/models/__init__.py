@@ -3,4 +3,5 @@ from . import fidolix  # noqa: F401
 from . import kedelorn  # noqa: F401
 from . import llama  # noqa: F401
 from . import povusun  # noqa: F401
+from . import tobozen  # noqa: F401
 from . import zepavik  # noqa: F401

@@ -162,14 +162,17 @@ class Kernels:
         return (_ptr(stats.scaled), _ptr(gamma), _ptr(stats.partials), stats.partials.shape[1], _ptr(stats.row_scale),
                 ctypes.c_float(stats.next_norm.spec.eps), _NULL if stats.consumer_sums else _ptr(stats.counter))
 
-    def rmsnorm(self, x, gamma, eps: float, out, rows=None):
-        """out[r, :] = rmsnorm(x[rows[r] or r, :]) * gamma, in the compute dtype."""
+    def rmsnorm(self, x, gamma, eps: float, out, rows=None, groups: int = 1):
+        """out[r, :] = rmsnorm(x[rows[r] or r, :]) * gamma, in the compute dtype.  ``groups`` > 1: the row in that many
+        equal parts, each divided by its own root mean square."""
         self._want(x, torch.float32, "x"); self._want(gamma, torch.float32, "gamma")
         self._want(out, self.dtype, "out")
         hidden = x.shape[-1]
         n_rows = out.shape[0]
         if gamma.numel() != hidden or out.shape[-1] != hidden:
             raise KernelError("rmsnorm: shapes do not agree")
+        if groups < 1 or hidden % groups:
+            raise KernelError("rmsnorm: the groups must split a row into equal parts")
         if rows is not None:
             self._want(rows, torch.int32, "rows")
             if rows.numel() != n_rows:
@@ -177,7 +180,7 @@ class Kernels:
         elif x.shape[0] != n_rows:
             raise KernelError("rmsnorm: shapes do not agree")
         self._check(self.lib.skv_rmsnorm(_ptr(x), _ptr(gamma), ctypes.c_float(eps), _ptr(out), _ptr(rows),
-                                         n_rows, hidden, _stream()), "rmsnorm")
+                                         n_rows, hidden, int(groups), _stream()), "rmsnorm")
 
     def linear(self, a, w, out, mode: int = MODE_STORE, activation: str = "silu", flag=None, stats=None,
                activation_param: float = 0.0):
@@ -911,14 +914,26 @@ class Kernels:
         self._check(self.lib.skv_gather_rows(_ptr(a), a.stride(0), _ptr(rows), _ptr(out), out.shape[0], out.shape[1],
                                              _stream()), "gather_rows")
 
+    def scatter_rows(self, a, place, weights, out):
+        """``out[place[t, k]] = a[t] * weights[t, k]`` for every (token, choice) pair: the tokens' rows in sorted order,
+        weighted, for experts whose weights multiply their inputs."""
+        self._want(a, self.dtype, "a"); self._want(out, self.dtype, "out"); self._want(place, torch.int32, "place")
+        self._want(weights, torch.float32, "weights")
+        n, top = place.shape
+        if tuple(weights.shape) != (n, top) or a.shape[0] != n or tuple(out.shape) != (n * top, a.shape[1]):
+            raise KernelError("scatter_rows: shapes do not agree")
+        self._check(self.lib.skv_scatter_rows(_ptr(a), _ptr(place), _ptr(weights), top, _ptr(out), n * top, a.shape[1],
+                                              _stream()), "scatter_rows")
+
     def expert_rows_sorted_first(self, hidden: int) -> bool:
         """True if ``expert_linear`` is faster on rows that lie in sorted order (``gather_rows`` first): the bfloat16
         build's tensor-core form wants neighbouring rows of whole 16 bytes."""
         return self.dtype == torch.bfloat16 and hidden % 8 == 0
 
     def expert_linear(self, a, w, offsets, out, rows=None, activation: Optional[str] = None, flag=None,
-                      gated: bool = False):
-        """(``gated``: ``w`` is ``[experts, 2 N, K]`` in tiles of 8 gate rows and their 8 up rows, as ``pack_gate_up``
+                      gated: bool = False, activation_param: float = 0.0):
+        """(``activation_param``: the number of a parametric activation, which gated experts may have.)
+        (``gated``: ``w`` is ``[experts, 2 N, K]`` in tiles of 8 gate rows and their 8 up rows, as ``pack_gate_up``
         lays them out, and ``out[p] = act(gate_e . a) * (up_e . a)``.)
         ``out[p] = act(w[e] . a[row(p)])`` for every sorted pair p of expert e (``offsets`` from ``sort_by_expert``);
         ``w`` ``[experts, N, K]``; ``row(p) = rows[p]`` (the first projection gathers its input from the tokens) or p.
@@ -938,21 +953,25 @@ class Kernels:
             self._want(rows, torch.int32, "rows")
             if rows.numel() != pairs:
                 raise KernelError("expert_linear: one row index per pair is needed")
-        if activation is not None and (activation not in ACTIVATIONS or activation in PARAMETRIC_ACTIVATIONS):
+        if activation is not None and (activation not in ACTIVATIONS or (activation in PARAMETRIC_ACTIVATIONS and not gated)):
             raise KernelError(f"expert_linear: activation '{activation}' is not supported")
         self._check(self.lib.skv_expert_linear(
             _ptr(a), a.stride(0), a.shape[0], _ptr(rows), _ptr(w), _ptr(offsets), _ptr(out),
-            int(out.dtype == torch.float32), pairs, experts, N, K, ACTIVATIONS[activation] if activation is not None else -1,
+            int(out.dtype == torch.float32), pairs, experts, N, K,
+            activation_word(activation, activation_param) if activation is not None else ctypes.c_longlong(-1),
             int(bool(gated)), _ptr(flag if flag is not None else self.error_flag), _stream()), "expert_linear")
 
     def combine_experts(self, results, place, weights, shared, share, x, add: bool = True):
         """``x[t] (+)= sum_k weights[t, k] * results[place[t, k]] + share[t] * shared[t]`` (float32; ``shared`` may be
-        None, ``share`` None counts as one); ``add`` false stores instead of adding."""
+        None, ``share`` None counts as one, and so does ``weights`` None); ``add`` false stores instead of adding."""
         self._want(results, torch.float32, "results"); self._want(place, torch.int32, "place")
-        self._want(weights, torch.float32, "weights"); self._want(x, torch.float32, "x")
+        self._want(x, torch.float32, "x")
+        if weights is not None:
+            self._want(weights, torch.float32, "weights")
         n, hidden = x.shape
         top = place.shape[1]
-        if results.shape[1] != hidden or results.shape[0] != n * top or tuple(weights.shape) != (n, top) or place.shape[0] != n:
+        if (results.shape[1] != hidden or results.shape[0] != n * top or place.shape[0] != n
+                or (weights is not None and tuple(weights.shape) != (n, top))):
             raise KernelError("combine_experts: shapes do not agree")
         if shared is not None:
             self._want(shared, torch.float32, "shared")
@@ -1113,6 +1132,148 @@ class Kernels:
         self._check(self.lib.skv_time_mix_finish(_ptr(o), _ptr(gate), o.shape[1], _ptr(norm), ctypes.c_float(eps),
                                                  ctypes.c_float(out_scale), _ptr(out), out.shape[1], n, int(heads),
                                                  int(dim), _stream()), "time_mix_finish")
+
+    # ---- attention's inputs behind a norm over all heads --------------------------------------
+    def normed_rotary(self, rows, q_out, k_cache, v_cache, positions, token_seq, block_table, num_heads: int,
+                      num_kv_heads: int, dim: int, vdim: int, block_size: int, eps: float = 0.0, q_weight=None,
+                      k_weight=None, cos_sin=None, rotated: int = 0, interleaved: bool = False, mix=None, first=None,
+                      keep=None, write_kv: bool = True):
+        """From float32 rows ``[q | k | v | ...]`` of a fused projection: one RMS norm with ``q_weight`` over all query
+        heads and one with ``k_weight`` over all key heads (None: no norm), rotary positions on the first ``rotated``
+        numbers of every head (``cos_sin`` ``[positions, rotated / 2, 2]``; pairs ``(2i, 2i + 1)`` if ``interleaved`` else
+        ``(i, i + rotated / 2)``), queries to ``q_out`` and keys and values to the cache.  ``mix`` (one float32 number on the
+        device) with ``first`` (float32 ``[tokens, kv_heads * vdim]``): the values are ``(1 - mix) v + mix first``; ``keep``
+        (the same shape) gets the values before that.  ``q_out`` and the caches may hold wider heads (multiples of a
+        common width), whose further numbers are set to zero."""
+        self._want(rows, torch.float32, "rows"); self._want(q_out, self.dtype, "q_out")
+        self._want(positions, torch.int32, "positions"); self._want(token_seq, torch.int32, "token_seq")
+        self._want(block_table, torch.int32, "block_table")
+        self._want(k_cache, self.dtype, "k_cache"); self._want(v_cache, self.dtype, "v_cache")
+        n = rows.shape[0]
+        q_width, v_width = k_cache.shape[-1], v_cache.shape[-1]
+        if (rows.shape[1] < num_heads * dim + num_kv_heads * (dim + vdim) or tuple(q_out.shape) != (n, num_heads * q_width)
+                or positions.numel() != n or token_seq.numel() != n or q_width < dim or v_width < vdim
+                or tuple(k_cache.shape[1:3]) != (num_kv_heads, block_size) or tuple(v_cache.shape[1:3]) != (num_kv_heads, block_size)):
+            raise KernelError("normed_rotary: shapes do not agree")
+        for name, weight, width in (("q_weight", q_weight, num_heads * dim), ("k_weight", k_weight, num_kv_heads * dim), ("mix", mix, 1)):
+            if weight is not None:
+                self._want(weight, torch.float32, name)
+                if weight.numel() != width:
+                    raise KernelError(f"normed_rotary: {name} must hold {width} numbers")
+        for name, values in (("first", first), ("keep", keep)):
+            if values is not None:
+                self._want(values, torch.float32, name)
+                if tuple(values.shape) != (n, num_kv_heads * vdim):
+                    raise KernelError(f"normed_rotary: {name} must be [tokens, kv_heads * vdim]")
+        if (mix is None) != (first is None):
+            raise KernelError("normed_rotary: mixed values need the share and the other values")
+        if rotated > 0:
+            self._want(cos_sin, torch.float32, "cos_sin")
+            if cos_sin.dim() != 3 or cos_sin.shape[1] * 2 != rotated or rotated > dim:
+                raise KernelError("normed_rotary: the rotation's table must be [positions, rotated / 2, 2]")
+        self._check(self.lib.skv_normed_rotary(
+            _ptr(rows), rows.shape[1], _ptr(q_weight), _ptr(k_weight), ctypes.c_float(eps),
+            _ptr(cos_sin if rotated > 0 else None), int(rotated), int(bool(interleaved)), _ptr(mix), _ptr(first), _ptr(keep),
+            _ptr(positions), _ptr(token_seq), _ptr(block_table), block_table.shape[1], _ptr(q_out), _ptr(k_cache),
+            _ptr(v_cache), n, num_heads, num_kv_heads, dim, vdim, q_width, v_width, block_size, int(bool(write_kv)),
+            _stream()), "normed_rotary")
+
+    # ---- linear attention with a matrix state ---------------------------------------------------
+    def linear_state_scratch(self, n_seqs: int, max_q_len: int, heads: int, dim: int, vdim: int) -> int:
+        """Floats of scratch ``linear_state`` needs for a step whose longest sequence brings ``max_q_len`` tokens."""
+        self.lib.skv_linear_state_scratch.restype = ctypes.c_longlong
+        return int(self.lib.skv_linear_state_scratch(int(n_seqs), int(max_q_len), int(heads), int(dim), int(vdim)))
+
+    def linear_state(self, rows, q_at: int, k_at: int, v_at: int, out, state, step_meta, heads: int, groups: int, dim: int,
+                     vdim: int, max_q_len: int, decay=None, log_decay=None, key_scale=None, skip=None, silu: bool = False,
+                     scratch=None, state_offset: int = 0):
+        """Per head ``S <- d S + c k v^T`` and ``out = S^T q + skip v`` over a packed step (all float32).  ``rows`` hold
+        ``groups`` query and key heads of ``dim`` numbers from columns ``q_at`` and ``k_at`` and ``heads`` value heads of
+        ``vdim`` from ``v_at`` (``silu``: passed through silu as they are read).  The decay d is ``decay[head]`` or
+        ``exp(log_decay[token, head])``, the factor c ``key_scale[token, head]`` or 1.  ``out`` ``[tokens, heads * vdim]``.
+        ``state``: float32 ``[slots, floats]``, S twice from ``state_offset`` on (in the half of the last written position's
+        parity).  ``scratch``: ``linear_state_scratch`` floats."""
+        for name, tensor, shape in (("decay", decay, (heads,)), ("skip", skip, (heads,)),
+                                    ("log_decay", log_decay, (rows.shape[0], heads)), ("key_scale", key_scale, (rows.shape[0], heads))):
+            if tensor is not None:
+                self._want(tensor, torch.float32, name)
+                if tuple(tensor.shape) != shape:
+                    raise KernelError(f"linear_state: {name} must be {list(shape)}")
+        self._want(rows, torch.float32, "rows"); self._want(out, torch.float32, "out")
+        n, n_seqs = rows.shape[0], step_meta[3].numel()
+        if (decay is None) == (log_decay is None):
+            raise KernelError("linear_state: one decay per head, or one logarithm per token and head")
+        if tuple(out.shape) != (n, heads * vdim) or groups <= 0 or heads % groups or step_meta[0].numel() != n:
+            raise KernelError("linear_state: shapes do not agree")
+        need = self.linear_state_scratch(n_seqs, max_q_len, heads, dim, vdim)
+        if need:
+            self._want(scratch, torch.float32, "scratch")
+            if scratch.numel() < need:
+                raise KernelError("linear_state: the scratch for the chunks is too small")
+        self._check(self.lib.skv_linear_state(
+            _ptr(rows), rows.shape[1], int(q_at), int(k_at), int(v_at), int(bool(silu)), _ptr(decay), _ptr(log_decay),
+            _ptr(key_scale), _ptr(skip), _ptr(out), _ptr(scratch if need else None), n, n_seqs, heads, groups, dim, vdim,
+            int(max_q_len), *self._state_args(step_meta, state, state_offset), _stream()), "linear_state")
+        if max_q_len > 1:
+            Kernels.launches += 2              # (the chunks' sums, the walk over the chunks, the outputs)
+
+    def mamba2_step(self, rows, conv_w, conv_b, dt_at: int, dt_bias, a_log, skip, out, state, step_meta, heads: int,
+                    groups: int, dim: int, vdim: int, state_offset: int, ring_offset: int):
+        """One token a sequence of a Mamba-2 mixer between its projections: the convolution with bias and silu on the rows'
+        first columns ``[values | keys | queries]``, the step size ``dt = softplus(rows[:, dt_at:] + dt_bias)``, then
+        ``linear_state`` with decay ``exp(-exp(a_log) dt)``, factor dt and ``skip``.  ``state`` holds S twice from
+        ``state_offset`` and the convolution's last inputs ``[taps, channels]`` from ``ring_offset``."""
+        self._want(rows, torch.float32, "rows"); self._want(out, torch.float32, "out"); self._want(conv_w, torch.float32, "conv_w")
+        n, channels = rows.shape[0], heads * vdim + 2 * groups * dim
+        for name, tensor, size in (("conv_b", conv_b, channels), ("dt_bias", dt_bias, heads), ("a_log", a_log, heads), ("skip", skip, heads)):
+            self._want(tensor, torch.float32, name)
+            if tensor.numel() != size:
+                raise KernelError(f"mamba2_step: {name} must hold {size} numbers")
+        if (conv_w.dim() != 2 or conv_w.shape[0] != channels or tuple(out.shape) != (n, heads * vdim)
+                or rows.shape[1] < channels or step_meta[3].numel() != n):
+            raise KernelError("mamba2_step: shapes do not agree")
+        args = self._state_args(step_meta, state, state_offset)
+        self._check(self.lib.skv_mamba2_step(
+            _ptr(rows), rows.shape[1], _ptr(conv_w), _ptr(conv_b), conv_w.shape[1], int(dt_at), _ptr(dt_bias), _ptr(a_log),
+            _ptr(skip), _ptr(out), n, heads, groups, dim, vdim, *args, ctypes.c_longlong(ring_offset), _stream()), "mamba2_step")
+
+    def conv_silu(self, rows, conv_w, conv_b, out, step_meta, state, ring_offset: int = 0):
+        """``out = silu(conv_b + causal convolution over time)`` of the rows' first columns (float32, one channel each);
+        what lies before the step comes from the ring ``[taps, channels]`` at ``ring_offset`` of a slot's state, which
+        ``short_conv_remember`` writes."""
+        self._want(rows, torch.float32, "rows"); self._want(out, torch.float32, "out")
+        self._want(conv_w, torch.float32, "conv_w"); self._want(conv_b, torch.float32, "conv_b")
+        n, channels = out.shape
+        if conv_w.dim() != 2 or conv_w.shape[0] != channels or conv_b.numel() != channels or rows.shape[0] != n or rows.shape[1] < channels:
+            raise KernelError("conv_silu: shapes do not agree")
+        self._check(self.lib.skv_conv_silu(
+            _ptr(rows), rows.shape[1], _ptr(conv_w), _ptr(conv_b), channels, conv_w.shape[1], _ptr(out), n,
+            *self._state_args(step_meta, state, ring_offset), _stream()), "conv_silu")
+
+    def step_sizes(self, rows, dt_at: int, dt_bias, a_log, dt, log_decay):
+        """``dt = softplus(rows[:, dt_at:dt_at + heads] + dt_bias)``, ``log_decay = -exp(a_log) dt`` (float32)."""
+        for name, tensor in (("rows", rows), ("dt_bias", dt_bias), ("a_log", a_log), ("dt", dt), ("log_decay", log_decay)):
+            self._want(tensor, torch.float32, name)
+        n, heads = dt.shape
+        if tuple(log_decay.shape) != (n, heads) or rows.shape[0] != n or rows.shape[1] < dt_at + heads or \
+                dt_bias.numel() != heads or a_log.numel() != heads:
+            raise KernelError("step_sizes: shapes do not agree")
+        self._check(self.lib.skv_step_sizes(_ptr(rows), rows.shape[1], int(dt_at), _ptr(dt_bias), _ptr(a_log), heads, n, _ptr(dt),
+                                            _ptr(log_decay), _stream()), "step_sizes")
+
+    def gated_norm(self, y, gate, gate_stride: int, weight, groups: int, eps: float, gate_first: bool, out):
+        """An RMS norm of float32 rows in ``groups`` equal parts, times ``weight``, with a gate on every number:
+        ``gate_first``: ``norm(y * silu(gate))``, else ``norm(y) * sigmoid(gate)``.  ``gate``: a float32 view whose rows are
+        ``gate_stride`` numbers apart.  ``out`` in the compute dtype; columns beyond the row are set to zero."""
+        self._want(y, torch.float32, "y"); self._want(weight, torch.float32, "weight"); self._want(out, self.dtype, "out")
+        n, width = y.shape
+        if gate.dtype != torch.float32 or not gate.is_cuda or gate.stride(-1) != 1 or gate.shape[0] != n or gate.stride(0) != gate_stride:
+            raise KernelError("gated_norm: the gate must be float32 rows on the GPU")
+        if weight.numel() != width or groups < 1 or width % groups or out.shape[0] != n or out.shape[1] < width:
+            raise KernelError("gated_norm: shapes do not agree")
+        self._check(self.lib.skv_gated_norm(_ptr(y), _ptr(gate), int(gate_stride), _ptr(weight), width, int(groups),
+                                            ctypes.c_float(eps), int(bool(gate_first)), _ptr(out), out.shape[1], n, _stream()),
+                    "gated_norm")
 
     def scale_inplace(self, x, factor: float):
         self._want(x, torch.float32, "x")

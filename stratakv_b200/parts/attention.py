@@ -70,6 +70,41 @@ def _residual_stats(step):
     return None if getattr(step, "store_branch", False) else step.residual_stats
 
 
+def attend_with_sink(step, rt, q, ctx, k_cache, v_cache, table, heads: int, kv_heads: int, dim: int, vdim: int,
+                     scale: float, window: int = 0, sink=None) -> None:
+    """Attention of finished queries ``q`` over the cache, which holds the step's keys and values already, with a sink per
+    head in the softmax's denominator (``sink`` float32 ``[heads]`` or None).  bfloat16 heads of 64 or 128 numbers with
+    values as wide: prompts on the tensor-core kernel; one token a sequence on the split kernel (the query heads of a key
+    head as rows of a tensor-core product, the context in pieces, the sink in the merge).  Everything else: the kernel
+    with run-time head sizes, a one-token step's keys cut into parts that run side by side."""
+    n, block_size = q.shape[0], step.cache.block_size
+    built = (rt.dtype == torch.bfloat16 and rt.device.type == "cuda" and dim == vdim and dim in (64, 128)
+             and ctx.shape[1] == heads * vdim)
+    if (built and step.max_q_len > 32 and block_size & (block_size - 1) == 0 and block_size >= 16
+            and step.n_seqs * -(-step.max_q_len // 128) <= 65535 and rt.kernels(dim).has_attention_prefill_tc()):
+        rt.kernels(dim).attention_prefill_tc(q, k_cache, v_cache, table, step.cu_q, step.ctx_after, ctx, step.max_q_len,
+                                             heads, kv_heads, dim, block_size, scale, window, sink=sink)
+        return
+    splits, scratch_o, scratch_ml = 1, None, None
+    decode = step.is_decode and built and block_size % 16 == 0
+    if step.is_decode:
+        keys = min(step.max_ctx, window) if window > 0 else step.max_ctx
+        if decode:
+            splits = decode_splits(n, kv_heads * (-(-(heads // kv_heads) // 16)), keys, rt.sm_count)
+        else:
+            splits = max(1, min(-(-rt.sm_count * 32 // (n * heads)), -(-keys // 64), 64))
+        if splits > 1:
+            scratch_o = rt.workspace.get("attn_split_o", (n * heads * splits * vdim,), torch.float32)
+            scratch_ml = rt.workspace.get("attn_split_ml", (n * heads * splits * 2,), torch.float32)
+    if decode:
+        rt.kernels(dim).attention_decode(q, k_cache, v_cache, table, step.ctx_after, ctx, heads, kv_heads, dim, block_size,
+                                         scale, window, splits, scratch_o, scratch_ml, sink=sink)
+        return
+    rt.kernels().attention_general(q, k_cache, v_cache, table, step.positions, step.token_seq, ctx, heads, kv_heads, dim,
+                                   vdim, block_size, scale, window, sink=sink, splits=splits, scratch_o=scratch_o,
+                                   scratch_ml=scratch_ml)
+
+
 class PagedAttention(Mixer):
     graph_safe = True
     folds_norm = True

@@ -24,7 +24,8 @@ class TensorRequest:
     """A checkpoint tensor a part needs.  ``init`` tells the random-weights mode
     how to fill it: ``normal`` is N(0, std), ``around_one`` is 1 + N(0, std), ``positive`` is
     0.05 + |N(0, 0.5)|, ``around_identity`` the identity matrix + N(0, std), ``conv_taps`` N(0, 1) / taps,
-    ``unit_interval`` sigmoid(N(0, 1)), ``decay_logit`` N(-3, 1.5), ``half_normal`` |N(0, 0.5)|."""
+    ``unit_interval`` sigmoid(N(0, 1)), ``decay_logit`` N(-3, 1.5), ``half_normal`` |N(0, 0.5)|,
+    ``log_rate`` the logarithm of a rate between 1 and 16."""
     shape: Tuple[int, ...]
     init: str = "normal"
 

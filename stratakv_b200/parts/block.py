@@ -51,15 +51,19 @@ def foldable(norm, consumer):
 
 
 def pre_norm(layer: Layer, step, x, entry) -> None:
-    if layer.mixer_norm is None or layer.mixer is None or layer.ffn_norm is None or layer.ffn is None:
-        raise ValueError("the pre_norm arrangement needs a norm and a mixer, and a norm and a feed-forward")
+    if layer.mixer_norm is None or layer.mixer is None:
+        raise ValueError("the pre_norm arrangement needs a norm and a mixer")
+    if layer.ffn is not None and layer.ffn_norm is None:
+        raise ValueError("the pre_norm arrangement needs a norm for its feed-forward")
     stats = step.residual_stats
     h = _normed(layer.mixer_norm, layer.mixer, step, x)
     if stats is not None:
-        stats.expect(foldable(layer.ffn_norm, layer.ffn))
+        stats.expect(foldable(layer.ffn_norm, layer.ffn) if layer.ffn is not None else step.norm_after_layer)
     layer.mixer.forward(step, h, x, entry.cache, entry.writes_cache)
     if stats is not None and not layer.mixer.folds_norm:
         stats.invalidate()
+    if layer.ffn is None:
+        return
     h = _normed(layer.ffn_norm, layer.ffn, step, x)
     if stats is not None:
         stats.expect(step.norm_after_layer)
@@ -92,7 +96,8 @@ def parallel(layer: Layer, step, x, entry) -> None:
 
 def _fusable(norm):
     """True if the kernels that add to the stream can also apply this norm to their result (a plain RMS norm)."""
-    return norm is not None and getattr(norm.spec, "kind", None) == "rmsnorm" and hasattr(norm, "gamma")
+    return (norm is not None and getattr(norm.spec, "kind", None) == "rmsnorm" and hasattr(norm, "gamma")
+            and getattr(norm, "groups", 1) == 1)
 
 
 def _branch(part, step, h, shape, *cache_args):

@@ -21,7 +21,7 @@ from __future__ import annotations
 import torch
 
 from .. import ops as _ops
-from .attention import _residual_mode, _residual_stats
+from .attention import _residual_mode, _residual_stats, attend_with_sink
 from .base import CacheRequest, Mixer, TensorRequest
 from .position import RotaryTable
 from .registry import register_mixer
@@ -118,53 +118,9 @@ class ConvAttention(Mixer):
         if writes_cache:
             ops.short_conv_remember(fused, self.bias, self.channels, s.taps, step.n_seqs, meta, state, self.state_offset)
         ctx = rt.workspace.get("attn_ctx", (n, self.ctx_width), rt.dtype)
-        self._attend(step, q, ctx, k_cache, v_cache, table)
+        attend_with_sink(step, rt, q, ctx, k_cache, v_cache, table, s.num_heads, s.num_kv_heads, s.head_dim, s.head_dim,
+                         s.scale, s.window, self.sink)
         ops.linear(ctx, self.w_o, x, _residual_mode(step), stats=_residual_stats(step))
-
-    def _tensor_core_prompt(self, step) -> bool:
-        s, rt = self.spec, self.rt
-        block_size = step.cache.block_size
-        return (rt.dtype == torch.bfloat16 and rt.device.type == "cuda" and s.head_dim in (64, 128)
-                and self.ctx_width == self.q_dim and step.max_q_len > 32 and block_size & (block_size - 1) == 0
-                and block_size >= 16 and step.n_seqs * -(-step.max_q_len // 128) <= 65535
-                and rt.kernels(s.head_dim).has_attention_prefill_tc())
-
-    def _attend(self, step, q, ctx, k_cache, v_cache, table):
-        s, rt = self.spec, self.rt
-        n = q.shape[0]
-        block_size = step.cache.block_size
-        if self._tensor_core_prompt(step):
-            rt.kernels(s.head_dim).attention_prefill_tc(
-                q, k_cache, v_cache, table, step.cu_q, step.ctx_after, ctx, step.max_q_len, s.num_heads, s.num_kv_heads,
-                s.head_dim, block_size, s.scale, s.window, sink=self.sink)
-            return
-        if (step.is_decode and rt.dtype == torch.bfloat16 and rt.device.type == "cuda" and s.head_dim in (64, 128)
-                and self.ctx_width == self.q_dim and block_size % 16 == 0):
-            # one token a sequence at a head size the split kernel is built for: the query heads of a key head as
-            # rows of a tensor-core product, the context in pieces, the sink in the merge
-            from .attention import decode_splits
-            blocks_per_seq = s.num_kv_heads * (-(-(s.num_heads // s.num_kv_heads) // 16))
-            keys = min(step.max_ctx, s.window) if s.window > 0 else step.max_ctx
-            splits = decode_splits(n, blocks_per_seq, keys, rt.sm_count)
-            scratch_o = scratch_ml = None
-            if splits > 1:
-                scratch_o = rt.workspace.get("attn_split_o", (n * s.num_heads * splits * s.head_dim,), torch.float32)
-                scratch_ml = rt.workspace.get("attn_split_ml", (n * s.num_heads * splits * 2,), torch.float32)
-            rt.kernels(s.head_dim).attention_decode(q, k_cache, v_cache, table, step.ctx_after, ctx, s.num_heads,
-                                                    s.num_kv_heads, s.head_dim, block_size, s.scale, s.window, splits,
-                                                    scratch_o, scratch_ml, sink=self.sink)
-            return
-        splits, scratch_o, scratch_ml = 1, None, None
-        if step.is_decode:
-            # few tokens over long contexts: each (token, head)'s visible keys in parts that run side by side
-            keys = min(step.max_ctx, s.window) if s.window > 0 else step.max_ctx
-            splits = max(1, min(-(-rt.sm_count * 32 // (n * s.num_heads)), -(-keys // 64), 64))
-            if splits > 1:
-                scratch_o = rt.workspace.get("attn_split_o", (n * s.num_heads * splits * s.head_dim,), torch.float32)
-                scratch_ml = rt.workspace.get("attn_split_ml", (n * s.num_heads * splits * 2,), torch.float32)
-        rt.kernels().attention_general(q, k_cache, v_cache, table, step.positions, step.token_seq, ctx, s.num_heads,
-                                       s.num_kv_heads, s.head_dim, s.head_dim, block_size, s.scale, s.window,
-                                       sink=self.sink, splits=splits, scratch_o=scratch_o, scratch_ml=scratch_ml)
 
 
 register_mixer("conv_attention", ConvAttention)

@@ -16,6 +16,14 @@ class RMSNorm(Norm):
     graph_safe = True
     folds_norm = True
 
+    def __init__(self, spec, runtime):
+        super().__init__(spec, runtime)
+        self.groups = getattr(spec, "groups", 1)
+        if self.groups < 1 or spec.size % self.groups:
+            raise ValueError(f"rmsnorm: {spec.size} numbers do not split into {self.groups} equal groups")
+        if self.groups > 1:
+            self.folds_norm = False                   # (a factor per part does not commute with a projection)
+
     @classmethod
     def expected_tensors(cls, spec):
         around_zero = bool(getattr(spec, "weight_offset", 0.0))
@@ -34,7 +42,10 @@ class RMSNorm(Norm):
         n_rows = x.shape[0] if rows is None else rows.numel()
         if out is None:
             out = self.rt.workspace.get(name, (n_rows, self.spec.size), self.rt.dtype)
-        self.rt.kernels().rmsnorm(x, self.gamma, self.spec.eps, out, rows)
+        if self.groups > 1:
+            self.rt.kernels().rmsnorm(x, self.gamma, self.spec.eps, out, rows, groups=self.groups)
+        else:
+            self.rt.kernels().rmsnorm(x, self.gamma, self.spec.eps, out, rows)
         return out
 
 

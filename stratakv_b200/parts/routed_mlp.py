@@ -8,6 +8,9 @@ shared expert if the layer has one.
                                                                                the spec says `renormalize`)
       + sigmoid(shared.gate . h) * shared.down act(shared.up h)
 
+With ``spec.weigh_input`` the weights multiply the experts' inputs instead: ``y = sum over chosen e of
+expert_e(s_e * route_scale * h)``.
+
 An expert may be gated (``spec.gate_weights``): ``down_e (act(gate_e h) * (up_e h))``, gate and up rows packed in tiles as
 the dense gated feed-forward packs them.
 
@@ -33,14 +36,14 @@ class RoutedMlp(FeedForward):
 
     def __init__(self, spec, runtime):
         super().__init__(spec, runtime)
-        if spec.activation not in _ops.ACTIVATIONS or spec.activation in _ops.PARAMETRIC_ACTIVATIONS:
+        self.gated = getattr(spec, "gate_weights", None) is not None
+        if spec.activation not in _ops.ACTIVATIONS or (spec.activation in _ops.PARAMETRIC_ACTIVATIONS and not self.gated):
             raise ValueError(f"routed feed-forward: activation '{spec.activation}' is not supported")
         if not 0 < spec.top <= spec.experts or spec.experts > _ops.MAX_EXPERTS or spec.top > _ops.MAX_EXPERTS_PER_TOKEN:
             raise ValueError(f"routed feed-forward: {spec.top} of {spec.experts} experts is not supported (at most "
                              f"{_ops.MAX_EXPERTS_PER_TOKEN} of {_ops.MAX_EXPERTS})")
         if len(spec.up_weights) != spec.experts or len(spec.down_weights) != spec.experts:
             raise ValueError("routed feed-forward: one pair of tensor names per expert is needed")
-        self.gated = getattr(spec, "gate_weights", None) is not None
         if self.gated and len(spec.gate_weights) != spec.experts:
             raise ValueError("routed feed-forward: one gate tensor per expert is needed")
         self.score = getattr(spec, "score", "sigmoid")
@@ -53,6 +56,7 @@ class RoutedMlp(FeedForward):
         if runtime.dtype == torch.bfloat16 and spec.hidden_size % 8 != 0:
             raise ValueError(f"routed feed-forward: hidden size {spec.hidden_size} is not supported in bfloat16 "
                              "(rows of 16 bytes are needed: a multiple of 8); float32 takes any size")
+        self.weigh_input = getattr(spec, "weigh_input", False)
         self.padded = -(-spec.intermediate_size // 8) * 8
         self.shared_padded = -(-spec.shared.intermediate_size // 8) * 8 if spec.shared is not None else 0
 
@@ -122,13 +126,18 @@ class RoutedMlp(FeedForward):
         place = get("routed_place", (n, s.top), torch.int32)         # where each (token, choice) went
         ops.sort_by_expert(chosen, s.experts, offsets, order, place)
         hidden = get("routed_hidden", (pairs, self.padded), rt.dtype)
-        if ops.expert_rows_sorted_first(s.hidden_size):
+        gate = dict(activation=s.activation, gated=self.gated, activation_param=getattr(s, "activation_param", 0.0))
+        if self.weigh_input:
+            rows = get("routed_rows", (pairs, s.hidden_size), rt.dtype)
+            ops.scatter_rows(h, place, weights, rows)
+            ops.expert_linear(rows, self.w_up, offsets, hidden, **gate)
+        elif ops.expert_rows_sorted_first(s.hidden_size):
             # the tensor-core projection reads tiles of neighbouring rows: bring the tokens' rows into sorted order first
             gathered = get("routed_rows", (pairs, s.hidden_size), rt.dtype)
             ops.gather_rows(h, order, gathered)
-            ops.expert_linear(gathered, self.w_up, offsets, hidden, activation=s.activation, gated=self.gated)
+            ops.expert_linear(gathered, self.w_up, offsets, hidden, **gate)
         else:
-            ops.expert_linear(h, self.w_up, offsets, hidden, rows=order, activation=s.activation, gated=self.gated)
+            ops.expert_linear(h, self.w_up, offsets, hidden, rows=order, **gate)
         results = get("routed_results", (pairs, s.hidden_size), torch.float32)
         ops.expert_linear(hidden, self.w_down, offsets, results)
         shared_out = None
@@ -137,7 +146,7 @@ class RoutedMlp(FeedForward):
             ops.linear(h, self.shared_up, z, _ops.MODE_ACT, s.activation)
             shared_out = get("routed_shared", (n, s.hidden_size), torch.float32)
             ops.linear(z, self.shared_down, shared_out, _ops.MODE_STORE_F32)
-        ops.combine_experts(results, place, weights, shared_out, share, x, add=not getattr(step, "store_branch", False))
+        ops.combine_experts(results, place, None if self.weigh_input else weights, shared_out, share, x, add=not getattr(step, "store_branch", False))
 
 
 register_ffn("routed_mlp", RoutedMlp)

@@ -15,7 +15,8 @@ from typing import Any, Dict, List, Optional, Tuple
 
 @dataclass(frozen=True)
 class NormSpec:
-    """RMSNorm: ``y = x / sqrt(mean(x^2) + eps) * weight`` (``src/layers/rmsnorm.cpp:63-97``)."""
+    """RMSNorm: ``y = x / sqrt(mean(x^2) + eps) * weight`` (``src/layers/rmsnorm.cpp:63-97``).  ``groups`` > 1: the
+    vector in that many equal parts, each divided by its own root mean square."""
     size: int
     eps: float
     weight: str                      # tensor name
@@ -23,6 +24,7 @@ class NormSpec:
     # added to the stored weight when it is loaded: 1.0 for checkpoints that keep a norm's weight as its distance
     # from one (``y = x / rms * (1 + w)``)
     weight_offset: float = 0.0
+    groups: int = 1
 
 
 @dataclass(frozen=True)
@@ -220,6 +222,88 @@ class ConvAttentionSpec:
 
 
 @dataclass(frozen=True)
+class NormedAttentionSpec:
+    """Causal grouped-query attention with one RMS norm (``eps``) over all query heads together and one over all key heads
+    together before the heads are rotated (``q_norm`` ``[heads * head_dim]``, ``k_norm``; None: no norm), rotary positions
+    (``rope``), ``score = (q . k) scale``, and a softmax whose denominator also counts ``exp(sink_score)`` (one constant for
+    all heads, with no key and no value; None: none).
+
+    Values may be shared along the layers: a layer that ``keeps_values`` leaves its values for the layers after it in the
+    same step, and one with ``value_mix`` (a tensor name, one number m) has the values ``(1 - m) v + m kept`` and caches
+    those."""
+    hidden_size: int
+    num_heads: int
+    num_kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    eps: float
+    q_weight: str                    # [heads * dim, hidden]
+    k_weight: str                    # [kv_heads * dim, hidden]
+    v_weight: str                    # [kv_heads * vdim, hidden]
+    o_weight: str                    # [hidden, heads * vdim]
+    q_norm: Optional[str] = None
+    k_norm: Optional[str] = None
+    rope: Optional[RotarySpec] = None
+    sink_score: Optional[float] = None
+    keeps_values: bool = False
+    value_mix: Optional[str] = None
+    kind: str = "normed_attention"
+
+    @property
+    def kernel_head_dim(self) -> int:
+        """The head size whose compiled attention kernels serve this mixer, its heads padded to it; 0: none does."""
+        widest = max(self.dim, self.vdim)
+        return 64 if widest <= 64 else (128 if widest <= 128 else 0)
+
+
+@dataclass(frozen=True)
+class DecayAttentionSpec:
+    """Linear attention with a fixed decay per head (Lightning attention): ``q, k = silu(Wq h), silu(Wk h)`` (heads x
+    dim), ``v = silu(Wv h)`` (heads x vdim); per head ``S_t = decay S_(t-1) + k_t v_t^T`` (float32, zero at the start),
+    ``o_t = S_t^T q_t``; one RMS norm with ``norm`` over all heads together, times ``sigmoid(Wg h)``, then ``Wo``."""
+    hidden_size: int
+    num_heads: int
+    dim: int
+    vdim: int
+    decay: Tuple[float, ...]         # per head
+    eps: float
+    q_weight: str                    # [heads * dim, hidden]
+    k_weight: str
+    v_weight: str                    # [heads * vdim, hidden]
+    gate_weight: str                 # [heads * vdim, hidden]
+    norm: str                        # [heads * vdim]
+    o_weight: str                    # [hidden, heads * vdim]
+    kind: str = "decay_attention"
+
+
+@dataclass(frozen=True)
+class Mamba2Spec:
+    """The Mamba-2 mixer (state-space duality).  ``in_weight h = [z | x | B | C | dt]`` with ``inner = heads * vdim``
+    numbers for z and x, ``groups * state`` for B and C, one step size per head; x, B and C pass a causal convolution per
+    channel (``taps`` wide, with bias) and silu; ``dt = softplus(dt + dt_bias)``; per head, with its group's B and C,
+    ``S_t = exp(-exp(A_log) dt) S_(t-1) + dt B_t x_t^T`` (float32, zero at the start), ``y_t = S_t^T C_t + D x_t``;
+    ``y * silu(z)``, an RMS norm in ``norm_groups`` equal parts with ``norm``, then ``Wo``."""
+    hidden_size: int
+    num_heads: int
+    vdim: int
+    state: int
+    groups: int
+    taps: int
+    norm_groups: int
+    eps: float
+    in_weight: str                   # [2 inner + 2 groups * state + heads, hidden]
+    conv_weight: str                 # [inner + 2 groups * state, taps], the last column weighs the current token
+    conv_bias: str
+    dt_bias: str                     # [heads]
+    a_log: str                       # [heads]
+    skip: str                        # D, [heads]
+    norm: str                        # [inner]
+    o_weight: str                    # [hidden, inner]
+    kind: str = "mamba2"
+
+
+@dataclass(frozen=True)
 class TimeMixSpec:
     """Time mixing with a matrix state per head and a decay per token and key channel (the RWKV family).  With h' the
     token before's input (zeros for the first), every projection s of r, k, v, g, w reads ``h + (h' - h) mu_s``;
@@ -361,6 +445,9 @@ class RoutedMlpSpec:
     groups: int = 0
     keep_groups: int = 0
     renormalize_eps: float = 0.0     # added to the chosen scores' sum before ``renormalize`` divides by it
+    activation_param: float = 0.0    # the number of a parametric activation (gated experts)
+    # the weights multiply the experts' inputs and not their results: sum over chosen e of expert_e(s_e route_scale h)
+    weigh_input: bool = False
 
 
 @dataclass(frozen=True)
@@ -380,7 +467,7 @@ class LayerSpec:
     """One block: which norm, mixer and feed-forward, and how they are arranged.
 
     ``pre_norm``: ``x += mixer(norm1(x)); x += ffn(norm2(x))``
-    (``src/models/transformer_block.cpp:301-331``).
+    (``src/models/transformer_block.cpp:301-331``); ``ffn`` (with its norm) may be ``None``.
     ``parallel``: ``h = norm1(x); x += mixer(h) + ffn(h)``: one norm (``mixer_norm``), both branches read its
     output; ``ffn`` may be ``None``.
     ``sandwich``: ``x += post1(mixer(norm1(x))); x += post2(ffn(norm2(x)))``, then ``token_input`` if the layer

@@ -43,6 +43,8 @@ def random_tensor(name: str, request: TensorRequest, seed: int, std: float,
         values = values / std * 1.5 - 3.0
     elif request.init == "half_normal":        # non-negative numbers of order one half
         values = values.abs() / std * 0.5
+    elif request.init == "log_rate":           # the logarithm of a rate between 1 and 16
+        values = torch.log(1.0 + 15.0 * torch.sigmoid(values / std))
     elif request.init != "normal":
         raise ValueError(f"unknown init '{request.init}' for tensor {name}")
     return values.to(dtype)
