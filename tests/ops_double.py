@@ -25,9 +25,14 @@ class DoubleKernels:
         self.calls.append("embed")
         out.copy_(table[ids.long()].float())
 
-    def rmsnorm(self, x, gamma, eps, out, rows=None):
+    def rmsnorm(self, x, gamma, eps, out, rows=None, groups=1):
         self.calls.append("rmsnorm")
         src = x if rows is None else x[rows.long()]
+        if groups > 1:
+            parts = src.view(src.shape[0], groups, -1)
+            parts = parts / torch.sqrt((parts * parts).mean(dim=-1, keepdim=True) + eps)
+            out.copy_((parts.reshape(src.shape) * gamma).to(out.dtype))
+            return
         inv = 1.0 / torch.sqrt((src * src).mean(dim=-1, keepdim=True) + eps)
         out.copy_((src * inv * gamma).to(out.dtype))
 
@@ -321,7 +326,8 @@ class DoubleKernels:
     def expert_rows_sorted_first(self, hidden):
         return False
 
-    def expert_linear(self, a, w, offsets, out, rows=None, activation=None, flag=None, gated=False):
+    def expert_linear(self, a, w, offsets, out, rows=None, activation=None, flag=None, gated=False,
+                      activation_param=0.0):
         self.calls.append("expert_linear")
         for e in range(w.shape[0]):
             lo, hi = int(offsets[e]), int(offsets[e + 1])
@@ -331,14 +337,26 @@ class DoubleKernels:
             result = src.float() @ w[e].float().T
             if gated:                               # tiles of 8 gate rows and their 8 up rows
                 tiles = result.view(result.shape[0], -1, 2, 8)
-                result = (ACTIVATIONS[activation](tiles[:, :, 0]) * tiles[:, :, 1]).reshape(result.shape[0], -1)
+                gate, up = tiles[:, :, 0], tiles[:, :, 1]
+                if activation == "swiglu_clamp":
+                    gate = gate.clamp(max=activation_param)
+                    product = gate * torch.sigmoid(1.702 * gate) * (up.clamp(-activation_param, activation_param) + 1.0)
+                else:
+                    product = ACTIVATIONS[activation](gate) * up
+                result = product.reshape(result.shape[0], -1)
             elif activation is not None:
                 result = ACTIVATIONS[activation](result)
             out[lo:hi] = result.to(out.dtype)
 
+    def scatter_rows(self, a, place, weights, out):
+        self.calls.append("scatter_rows")
+        rows = (a.float()[:, None, :] * weights[:, :, None]).to(out.dtype)
+        out[place.reshape(-1).long()] = rows.reshape(-1, a.shape[1])
+
     def combine_experts(self, results, place, weights, shared, share, x, add=True):
         self.calls.append("combine_experts")
-        total = (results[place.long()] * weights[:, :, None]).sum(dim=1)
+        total = results[place.long()]
+        total = (total * weights[:, :, None] if weights is not None else total).sum(dim=1)
         if shared is not None:
             total = total + (shared * share[:, None] if share is not None else shared)
         if add:
@@ -515,6 +533,124 @@ class DoubleKernels:
         unit = heads_o / torch.sqrt((heads_o * heads_o).mean(dim=-1, keepdim=True) + eps)
         out.zero_()
         out[:, :heads * dim] = (unit.reshape(n, -1) * norm * gate * torch.sigmoid(gate) * out_scale).to(out.dtype)
+
+    def normed_rotary(self, rows, q_out, k_cache, v_cache, positions, token_seq, block_table, num_heads, num_kv_heads, dim,
+                      vdim, block_size, eps=0.0, q_weight=None, k_weight=None, cos_sin=None, rotated=0, interleaved=False,
+                      mix=None, first=None, keep=None, write_kv=True):
+        self.calls.append("normed_rotary")
+        n = rows.shape[0]
+        a, b, c = num_heads * dim, num_kv_heads * dim, num_kv_heads * vdim
+
+        def turned(x, weight, heads):
+            if weight is not None:
+                x = x / torch.sqrt((x * x).mean(dim=-1, keepdim=True) + eps) * weight
+            x = x.view(n, heads, dim)
+            out = x.clone()
+            if rotated:
+                cs = cos_sin[positions.long()]
+                co, sn = cs[:, None, :, 0], cs[:, None, :, 1]
+                even, odd = (slice(0, rotated, 2), slice(1, rotated, 2)) if interleaved else \
+                    (slice(0, rotated // 2), slice(rotated // 2, rotated))
+                out[..., even] = x[..., even] * co - x[..., odd] * sn
+                out[..., odd] = x[..., odd] * co + x[..., even] * sn
+            return out
+
+        q, k = turned(rows[:, :a], q_weight, num_heads), turned(rows[:, a:a + b], k_weight, num_kv_heads)
+        v = rows[:, a + b:a + b + c]
+        if keep is not None:
+            keep.copy_(v)
+        if mix is not None:
+            v = (1.0 - mix) * v + mix * first
+        v = v.reshape(n, num_kv_heads, vdim)
+        wide = q_out.view(n, num_heads, k_cache.shape[-1])
+        wide.zero_()
+        wide[..., :dim] = q.to(wide.dtype)
+        if not write_kv:
+            return
+        for t in range(n):
+            pos = int(positions[t])
+            block = int(block_table[int(token_seq[t]), pos // block_size])
+            for cache, value in ((k_cache, k[t]), (v_cache, v[t])):
+                row = cache[block, :, pos % block_size, :]
+                row.zero_()
+                row[:, :value.shape[-1]] = value.to(cache.dtype)
+
+    def linear_state_scratch(self, n_seqs, max_q_len, heads, dim, vdim):
+        return 0
+
+    def linear_state(self, rows, q_at, k_at, v_at, out, state, step_meta, heads, groups, dim, vdim, max_q_len, decay=None,
+                     log_decay=None, key_scale=None, skip=None, silu=False, scratch=None, state_offset=0):
+        self.calls.append("linear_state")
+        positions, token_seq, cu_q, slot_ids = step_meta
+        n = rows.shape[0]
+        act = ACTIVATIONS["silu"] if silu else (lambda z: z)
+        spread = lambda x: x.repeat_interleave(heads // groups, dim=1)
+        q = spread(act(rows[:, q_at:q_at + groups * dim]).view(n, groups, dim))
+        k = spread(act(rows[:, k_at:k_at + groups * dim]).view(n, groups, dim))
+        v = act(rows[:, v_at:v_at + heads * vdim]).view(n, heads, vdim)
+        if key_scale is not None:
+            k = k * key_scale[:, :, None]
+        d = decay.expand(n, heads) if decay is not None else torch.exp(log_decay)
+        size = heads * dim * vdim
+        for s in range(slot_ids.numel()):
+            first, last = int(cu_q[s]), int(cu_q[s + 1]) - 1
+            row = state[int(slot_ids[s])][state_offset:]
+            p_first = int(positions[first])
+            S = (row[((p_first - 1) & 1) * size:][:size].clone().view(heads, dim, vdim) if p_first > 0
+                 else torch.zeros(heads, dim, vdim))
+            for t in range(first, last + 1):
+                S = d[t][:, None, None] * S + k[t][:, :, None] * v[t][:, None, :]
+                o = torch.einsum("hnp,hn->hp", S, q[t])
+                out[t] = (o + skip[:, None] * v[t] if skip is not None else o).reshape(-1)
+            row[((p_first + last - first) & 1) * size:][:size] = S.reshape(size)
+
+    def conv_silu(self, rows, conv_w, conv_b, out, step_meta, state, ring_offset=0):
+        self.calls.append("conv_silu")
+        positions, token_seq, cu_q, slot_ids = step_meta
+        channels, taps = conv_w.shape
+        for t in range(rows.shape[0]):
+            seq, p = int(token_seq[t]), int(positions[t])
+            first = int(cu_q[seq])
+            y = conv_b.clone()
+            for j in range(taps):
+                back = taps - 1 - j
+                if p - back < 0:
+                    continue
+                if t - back >= first:
+                    u = rows[t - back, :channels]
+                else:
+                    ring = state[int(slot_ids[seq])][ring_offset:ring_offset + taps * channels].view(taps, channels)
+                    u = ring[(p - back) % taps]
+                y = y + conv_w[:, j] * u
+            out[t] = ACTIVATIONS["silu"](y)
+
+    def step_sizes(self, rows, dt_at, dt_bias, a_log, dt, log_decay):
+        self.calls.append("step_sizes")
+        dt.copy_(torch.nn.functional.softplus(rows[:, dt_at:dt_at + dt.shape[1]] + dt_bias))
+        log_decay.copy_(-torch.exp(a_log) * dt)
+
+    def mamba2_step(self, rows, conv_w, conv_b, dt_at, dt_bias, a_log, skip, out, state, step_meta, heads, groups, dim, vdim,
+                    state_offset, ring_offset):
+        self.calls.append("mamba2_step")
+        n, (channels, taps) = rows.shape[0], conv_w.shape
+        convolved = torch.zeros(n, channels)
+        self.conv_silu(rows, conv_w, conv_b, convolved, step_meta, state, ring_offset)
+        dt, log_decay = torch.zeros(n, heads), torch.zeros(n, heads)
+        self.step_sizes(rows, dt_at, dt_bias, a_log, dt, log_decay)
+        inner = heads * vdim
+        self.linear_state(convolved, inner + groups * dim, inner, 0, out, state, step_meta, heads, groups, dim, vdim, 1,
+                          log_decay=log_decay, key_scale=dt, skip=skip, state_offset=state_offset)
+        self.short_conv_remember(rows, None, channels, taps, n, step_meta, state, ring_offset)
+
+    def gated_norm(self, y, gate, gate_stride, weight, groups, eps, gate_first, out):
+        self.calls.append("gated_norm")
+        n, width = y.shape
+        g = gate[:, :width]
+        x = y * ACTIVATIONS["silu"](g) if gate_first else y
+        parts = x.view(n, groups, -1)
+        x = (parts / torch.sqrt((parts * parts).mean(dim=-1, keepdim=True) + eps)).reshape(n, width) * weight
+        out.zero_()
+        out[:, :width] = (x if gate_first else x * torch.sigmoid(g)).to(out.dtype)
 
     def scale_inplace(self, x, factor):
         x.mul_(factor)
