@@ -5,6 +5,8 @@
     python bench.py --design povusun [--layers 8]       (the Povusun decoder beside Llama: mixed layers, and each of its
                                                          three mixers alone)
     python bench.py --design fidolix [--layers 8]       (the Fidolix decoder beside Llama and beside the Kedelorn decoder)
+    python bench.py --design tobozen [--layers 9]       (the Tobozen decoder beside Llama and beside the nearest layers of the
+                                                         Kedelorn and Fidolix decoders: mixed layers, and each mixer alone)
     python bench.py --design kedelorn [--layers 8]      (the Kedelorn decoder beside Llama and beside Povusun's latent and
                                                          recurrent layers: mixed layers, and each of its two mixers alone)
 
@@ -425,8 +427,93 @@ def fidolix_arm(args) -> int:
     return 0
 
 
+def tobozen_config(size, layers, vocab, kinds):
+    """A Tobozen configuration at a size of DESIGN_SIZES whose layer i has the mixer ``kinds[i % len(kinds)]``.  The
+    attention layers have Llama's heads, key heads and head size, the whole head rotated, and mix their values.  The
+    Mamba-2 layers are twice as wide inside as the model, in heads of 64 with a state of 128, eight groups and four taps;
+    the Lightning layers have Llama's heads with keys and values of the head size.  Every layer has eight experts of which
+    two are chosen, each half as wide as Llama's feed-forward, so that a token passes through as many feed-forward weights
+    as in Llama.  The norms have two groups."""
+    from stratakv_b200.config import TobozenConfig
+    d, heads = size["head_dim"], size["heads"]
+    mlp = {"kind": "moe", "expert": {"ff": size["llama_ff"] // 2 // 64 * 64, "limit": 7.0}, "router": {"experts": 8, "top": 2}}
+    mixers = {
+        "attention": {"heads": heads, "kv_heads": size["kv_heads"], "dim": d, "vdim": d, "scale": d ** -0.5,
+                      "rot": {"dims": d, "base": 10000.0}, "v_mix": True},
+        "mamba2": {"heads": 2 * size["hidden"] // 64, "vdim": 64, "state": 128, "groups": 8, "conv": 4, "norm_groups": 8},
+        "lightning": {"heads": heads, "dim": d, "vdim": d,
+                      "decay": [1.0 - 2.0 ** (-5.0 - 3.0 * h / max(heads - 1, 1)) for h in range(heads)]}}
+    made = [{"type": kinds[i % len(kinds)], "mixer": mixers[kinds[i % len(kinds)]], "mlp": mlp} for i in range(layers)]
+    return TobozenConfig.from_dict({"architecture": "Tobozen", "vocab": vocab, "width": size["hidden"],
+                                    "norm": {"eps": 1e-5, "groups": 2}, "layers": made})
+
+
+def tobozen_arm(args) -> int:
+    """Prefill and decode of the Tobozen decoder beside the Llama decoder and beside the framework's nearest layers
+    (Kedelorn's retention, a matrix state with a decay per head; Fidolix's attention layer, with the same experts) at equal
+    layer sizes, random weights: a model that alternates its three kinds of layer, and one of each kind alone."""
+    import gc
+    import torch
+    from stratakv_b200.config import LlamaConfig
+    if not torch.cuda.is_available():
+        print("bench.py: no CUDA device")
+        return 1
+    layers, vocab, context, batch = args.layers or 9, 32000, args.context, args.batch
+    steps, warmup = max(args.steps, 1), max(args.warmup, 3)
+    peak = peaks()
+    sizes = {}
+    sampler = ClockSampler()
+    sampler.start()
+    for name, size in DESIGN_SIZES.items():
+        if args.sizes and name not in args.sizes.split(","):
+            continue
+        configs = {"llama": LlamaConfig.from_dict(dict(
+            TINYLLAMA, hidden_size=size["hidden"], intermediate_size=size["llama_ff"], num_hidden_layers=layers,
+            num_attention_heads=size["heads"], num_key_value_heads=size["kv_heads"], head_dim=size["head_dim"],
+            vocab_size=vocab, max_position_embeddings=context + 64)),
+            "kedelorn_retention_only": kedelorn_config(size, layers, vocab, ("retention",)),
+            "fidolix_attention_only": fidolix_config(size, layers, vocab, ("attention",)),
+            "tobozen": tobozen_config(size, layers, vocab, ("attention", "mamba2", "lightning")),
+            "tobozen_attention_only": tobozen_config(size, layers, vocab, ("attention",)),
+            "tobozen_mamba2_only": tobozen_config(size, layers, vocab, ("mamba2",)),
+            "tobozen_lightning_only": tobozen_config(size, layers, vocab, ("lightning",))}
+        only = [label for label in args.arms.split(",") if label] if args.arms else list(configs)
+        row = {}
+        for label in only:
+            engine = engine_of(configs[label], max(batch * (context + 64), PREFILL_TOKENS + 64), batch)
+            prefill_ms = time_prefill(engine, PREFILL_TOKENS, vocab)
+            decode_ms, launches, _ = time_decode(engine, batch, context - steps - warmup, steps, warmup, vocab)
+            weight_bytes = engine.model.weight_bytes()
+            kv_bytes = batch * context * engine.cache.bytes_per_token()
+            # (a recurrent layer reads one half of its state a step and writes the other)
+            state_bytes = batch * sum(engine.cache.state_bytes)
+            row[label] = {"prefill_tokens_per_s": PREFILL_TOKENS * 1000.0 / prefill_ms, "prefill_ms": prefill_ms,
+                          "decode_tokens_per_s": batch * 1000.0 / decode_ms, "decode_ms_per_step": decode_ms,
+                          "decode_hbm_frac": (weight_bytes + kv_bytes + state_bytes) / (decode_ms * 1e-3) / 1e9 / peak["hbm_gbs"],
+                          "weight_bytes": weight_bytes, "cache_bytes_per_token": engine.cache.bytes_per_token(),
+                          "state_bytes_per_step": state_bytes, "launches_in_timed_steps": launches}
+            engine.check_flags()
+            del engine
+            gc.collect()
+            torch.cuda.empty_cache()
+        if "llama" in row:
+            for label in row:
+                row[label]["prefill_ratio"] = row[label]["prefill_tokens_per_s"] / row["llama"]["prefill_tokens_per_s"]
+                row[label]["decode_ratio"] = row[label]["decode_tokens_per_s"] / row["llama"]["decode_tokens_per_s"]
+        sizes[name] = row
+    clocks = sampler.stop()
+    print(json.dumps({"design": "Tobozen", "beside": ["LlamaForCausalLM", "Kedelorn", "Fidolix"], "layers": layers, "vocab": vocab,
+                      "prefill_tokens": PREFILL_TOKENS, "decode_batch": batch, "context": context, "dtype": "bf16",
+                      "steps": steps, "warmup": warmup,
+                      "data": "synthetic: random N(0,0.02) weights, uniform random token ids", "peaks": peak,
+                      "clocks": clocks, "sizes": sizes}))
+    return 0
+
+
 def design_arm(args) -> int:
     """Prefill and decode of the Zepavik decoder and of the Llama decoder at equal layer sizes (random weights)."""
+    if args.design == "tobozen":
+        return tobozen_arm(args)
     if args.design == "fidolix":
         return fidolix_arm(args)
     if args.design == "povusun":
@@ -782,10 +869,10 @@ def main() -> int:
     parser.add_argument("--impl", default="ours", choices=["ours", "reference"])
     parser.add_argument("--skip-points", action="store_true", help="leave out batch 1 and 64 and the prefill")
     parser.add_argument("--context", type=int, default=CONTEXT, help="context at which the timed decode steps end")
-    parser.add_argument("--design", choices=["zepavik", "povusun", "kedelorn", "fidolix"],
+    parser.add_argument("--design", choices=["zepavik", "povusun", "kedelorn", "fidolix", "tobozen"],
                         help="measure this design beside the Llama decoder at equal layer sizes instead of the step benchmark")
     parser.add_argument("--sizes", default="", help="with --design: names of DESIGN_SIZES, with commas (default: all)")
-    parser.add_argument("--arms", default="", help="with --design kedelorn or fidolix: which models to time, with commas (default: all)")
+    parser.add_argument("--arms", default="", help="with --design kedelorn, fidolix or tobozen: which models to time, with commas (default: all)")
     parser.add_argument("--window", type=int, default=0, help="with --design: the design's window (default: the whole context)")
     parser.add_argument("--workload", choices=sorted(WORKLOADS),
                         help="a whole generation workload through Engine.generate instead of the step benchmark")

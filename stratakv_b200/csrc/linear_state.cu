@@ -92,11 +92,36 @@ linear_state_step_kernel(const float* __restrict__ rows, float* __restrict__ out
     float* partial = v + ((P + 3) & ~3);       // [LS_THREADS * VEC]
     __shared__ float head_numbers[2];          // the decay, the skip
     pdl_launch_dependents();
-    pdl_wait();
     const int head = blockIdx.x, s = blockIdx.y, g = head / (H / shape.groups);
     const int t = batch.cu_q[s], p = batch.positions[t];
     const float* row = rows + (size_t)t * shape.row_stride;
     float* slot = batch.state + (size_t)batch.slot_ids[s] * batch.state_stride;
+    const size_t half_size = (size_t)H * N * P;
+    const float* __restrict__ before = slot + batch.state_offset + (size_t)((p - 1) & 1) * half_size + (size_t)head * N * P;
+    float* __restrict__ after = slot + batch.state_offset + (size_t)(p & 1) * half_size + (size_t)head * N * P;
+    const int columns = P / VEC;                       // threads of a row of S
+    const int lanes = min(columns, LS_THREADS), per_pass = LS_THREADS / lanes;
+    const int r0 = threadIdx.x / lanes, c0 = threadIdx.x - r0 * lanes;
+    constexpr int AHEAD = 8;
+    float old[AHEAD][VEC];
+    auto fetch = [&](int n0, int c) {                  // this thread's next numbers of the state before the token
+#pragma unroll
+        for (int u = 0; u < AHEAD; ++u) {
+            const int n = n0 + u * per_pass;
+            const bool there = p > 0 && n < N && c < columns && r0 < per_pass;
+            if (VEC == 4) {
+                const float4 x = there ? *(const float4*)(before + (size_t)n * P + c * 4) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+                old[u][0] = x.x; old[u][1 % VEC] = x.y; old[u][2 % VEC] = x.z; old[u][3 % VEC] = x.w;
+            } else {
+                old[u][0] = there ? before[(size_t)n * P + c] : 0.0f;
+            }
+        }
+    };
+    // The step's metadata came with a copy in front of all its kernels, which also put everything that earlier steps
+    // launched behind it; the state before this token was written in an earlier step.  So the first part of it is fetched
+    // while the projection in front of this kernel still runs.
+    fetch(r0, c0);
+    pdl_wait();
     float scale = 1.0f;
     if (conv.conv_w) {
         float* ring = slot + conv.ring_offset;
@@ -126,12 +151,6 @@ linear_state_step_kernel(const float* __restrict__ rows, float* __restrict__ out
     if (threadIdx.x == 1) head_numbers[1] = decay.skip ? decay.skip[head] : 0.0f;
     __syncthreads();
     const float a = head_numbers[0];
-    const size_t half_size = (size_t)H * N * P;
-    const float* __restrict__ before = slot + batch.state_offset + (size_t)((p - 1) & 1) * half_size + (size_t)head * N * P;
-    float* __restrict__ after = slot + batch.state_offset + (size_t)(p & 1) * half_size + (size_t)head * N * P;
-    const int columns = P / VEC;                       // threads of a row of S
-    const int lanes = min(columns, LS_THREADS), per_pass = LS_THREADS / lanes;
-    const int r0 = threadIdx.x / lanes, c0 = threadIdx.x - r0 * lanes;
     for (int cb = 0; cb < columns; cb += lanes) {      // (more than one pass only where a row has more columns than threads)
         const int c = cb + c0;
         float acc[VEC];
@@ -141,19 +160,8 @@ linear_state_step_kernel(const float* __restrict__ rows, float* __restrict__ out
             float ve[VEC];
 #pragma unroll
             for (int e = 0; e < VEC; ++e) ve[e] = v[c * VEC + e];
-            constexpr int AHEAD = 8;
             for (int n0 = r0; n0 < N; n0 += per_pass * AHEAD) {
-                float old[AHEAD][VEC];
-#pragma unroll
-                for (int u = 0; u < AHEAD; ++u) {
-                    const int n = n0 + u * per_pass;
-                    if (VEC == 4) {
-                        const float4 x = p > 0 && n < N ? *(const float4*)(before + (size_t)n * P + c * 4) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-                        old[u][0] = x.x; old[u][1 % VEC] = x.y; old[u][2 % VEC] = x.z; old[u][3 % VEC] = x.w;
-                    } else {
-                        old[u][0] = p > 0 && n < N ? before[(size_t)n * P + c] : 0.0f;
-                    }
-                }
+                if (cb > 0 || n0 > r0) fetch(n0, c);
 #pragma unroll
                 for (int u = 0; u < AHEAD; ++u) {
                     const int n = n0 + u * per_pass;
@@ -184,25 +192,58 @@ linear_state_step_kernel(const float* __restrict__ rows, float* __restrict__ out
     }
 }
 
-// ---- longer steps ----------------------------------------------------------------------------------------------
-// l[j], c[j] and the sums of l behind every token of a chunk, in shared memory.  Called by the whole block.
-template <int CH>
-__device__ __forceinline__ void chunk_exponents(float* l, float* c, const LinearStateDecay& decay, int H, int head, int first,
-                                                int L) {
-    const float constant = decay.decay ? ls_log(decay.decay[head]) : 0.0f;
-    for (int j = threadIdx.x; j < CH; j += LS_THREADS) {
-        l[j] = j < L ? (decay.decay ? constant : decay.log_decay[(size_t)(first + j) * H + head]) : 0.0f;
-        c[j] = j < L ? (decay.key_scale ? decay.key_scale[(size_t)(first + j) * H + head] : 1.0f) : 0.0f;
-    }
-}
+// Where a thread stands in the 16 x 16 arrangement over a tile: a warp is four rows by eight columns of threads, so that a
+// 16-byte load a thread of either operand is one pass over shared memory (64 and 128 different bytes).
+__device__ __forceinline__ int tile_x() { return (threadIdx.x & 7) | ((threadIdx.x >> 5 & 1) << 3); }
+__device__ __forceinline__ int tile_y() { return (threadIdx.x >> 3 & 3) | ((threadIdx.x >> 6) << 2); }
 
-// exp of the sum of l over the tokens from .. to of a chunk (one product where the decay is one number per head)
-__device__ __forceinline__ float span_decay(const float* l, int from, int to, bool constant) {
-    if (to < from) return 1.0f;
-    if (constant) return expf((float)(to - from + 1) * l[0]);
-    float sum = 0.0f;
-    for (int i = from; i <= to; ++i) sum += l[i];
-    return expf(sum);
+// ---- longer steps ----------------------------------------------------------------------------------------------
+// The exponents of a chunk, in shared memory: l[j] and c[j] of every token, up_to[j] = exp(l_0 + .. + l_j) and
+// behind[j] = exp(l_(j+1) + .. + l_(L-1)).  Called by the first warp; a lane holds CH / 32 neighbouring tokens (one token, of
+// which half the lanes have none, where a chunk is 16).
+template <int CH>
+__device__ __forceinline__ void chunk_exponents(float* l, float* c, float* up_to, float* behind, const LinearStateDecay& decay,
+                                                int H, int head, int first, int L) {
+    constexpr int EACH = CH >= 32 ? CH / 32 : 1;
+    const int lane = threadIdx.x & 31;
+    const float constant = decay.decay ? ls_log(decay.decay[head]) : 0.0f;
+    float mine[EACH], key[EACH], total = 0.0f;
+#pragma unroll
+    for (int e = 0; e < EACH; ++e) {
+        const int j = lane * EACH + e;
+        mine[e] = j < L ? (decay.decay ? constant : decay.log_decay[(size_t)(first + j) * H + head]) : 0.0f;
+        key[e] = j < L ? (decay.key_scale ? decay.key_scale[(size_t)(first + j) * H + head] : 1.0f) : 0.0f;
+        total += mine[e];
+    }
+    float below = total, above = total;                       // sums over this lane and the lanes on either side of it
+#pragma unroll
+    for (int offset = 1; offset < 32; offset <<= 1) {
+        const float from_below = __shfl_up_sync(0xffffffffu, below, offset);
+        const float from_above = __shfl_down_sync(0xffffffffu, above, offset);
+        if (lane >= offset) below += from_below;
+        if (lane + offset < 32) above += from_above;
+    }
+    // (the neighbours' sums alone: never a difference of two sums)
+    float before = __shfl_up_sync(0xffffffffu, below, 1), after = __shfl_down_sync(0xffffffffu, above, 1);
+    if (lane == 0) before = 0.0f;
+    if (lane == 31) after = 0.0f;
+    if (lane * EACH >= CH) return;
+    float sum = before;
+#pragma unroll
+    for (int e = 0; e < EACH; ++e) {
+        const int j = lane * EACH + e;
+        l[j] = mine[e];
+        c[j] = key[e];
+        sum += mine[e];
+        up_to[j] = expf(decay.decay ? (float)(j + 1) * constant : sum);
+    }
+    sum = after;
+#pragma unroll
+    for (int e = EACH - 1; e >= 0; --e) {
+        const int j = lane * EACH + e;
+        behind[j] = j < L - 1 ? expf(decay.decay ? (float)(L - 1 - j) * constant : sum) : 1.0f;
+        sum += mine[e];
+    }
 }
 
 // sums [seqs][max_chunks][heads][dim][vdim], factors [seqs][max_chunks][heads].  Threads in 16 x 16, each with RN rows and
@@ -218,24 +259,23 @@ linear_state_sum_kernel(const float* __restrict__ rows, float* __restrict__ sums
     float* vs = ks + CH * TN;                             // [CH][64]
     float* l = vs + CH * 64;                              // [CH]
     float* c = l + CH;                                    // [CH]
-    float* w = c + CH;                                    // [CH]
+    float* up_to = c + CH;                                // [CH]
+    float* behind = up_to + CH;                           // [CH]
     pdl_launch_dependents();
     pdl_wait();
     const int chunk = blockIdx.x, head = blockIdx.y, s = blockIdx.z, g = head / (H / shape.groups);
     const int first = cu_q[s] + chunk * CH, L = min(CH, cu_q[s + 1] - first);
     if (L <= 0) return;
-    chunk_exponents<CH>(l, c, decay, H, head, first, L);
+    if (threadIdx.x < 32) chunk_exponents<CH>(l, c, up_to, behind, decay, H, head, first, L);
     __syncthreads();
-    const bool constant = decay.decay != nullptr;
-    for (int j = threadIdx.x; j < L; j += LS_THREADS) w[j] = c[j] * span_decay(l, j + 1, L - 1, constant);
     const size_t place = ((size_t)s * max_chunks + chunk) * H + head;
-    if (threadIdx.x == LS_THREADS - 1) factors[place] = span_decay(l, 0, L - 1, constant);
-    __syncthreads();
+    if (threadIdx.x == 0) factors[place] = up_to[L - 1];
     float* mine = sums + place * (size_t)N * P;
-    const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+    const int tx = tile_x(), ty = tile_y();
     const bool vec = ((shape.row_stride | shape.k_at | shape.v_at | N | P) & 3) == 0;
     for (int n0 = 0; n0 < N; n0 += TN) {
         if (vec) {
+#pragma unroll 4
             for (int idx = threadIdx.x; idx < L * (TN / 4); idx += LS_THREADS) {
                 const int j = idx / (TN / 4), n = (idx - j * (TN / 4)) * 4;
                 float4 x = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
@@ -243,13 +283,13 @@ linear_state_sum_kernel(const float* __restrict__ rows, float* __restrict__ sums
                     x = *(const float4*)(rows + (size_t)(first + j) * shape.row_stride + shape.k_at + g * N + n0 + n);
                     if (shape.silu) x = make_float4(ls_silu(x.x), ls_silu(x.y), ls_silu(x.z), ls_silu(x.w));
                 }
-                const float wj = w[j];
+                const float wj = c[j] * behind[j];
                 *(float4*)(ks + j * TN + n) = make_float4(x.x * wj, x.y * wj, x.z * wj, x.w * wj);
             }
         } else {
             for (int idx = threadIdx.x; idx < L * TN; idx += LS_THREADS) {
                 const int j = idx / TN, n = idx - j * TN;
-                ks[idx] = n0 + n < N ? ls_read(rows + (size_t)(first + j) * shape.row_stride + shape.k_at + g * N + n0 + n, shape.silu) * w[j] : 0.0f;
+                ks[idx] = n0 + n < N ? ls_read(rows + (size_t)(first + j) * shape.row_stride + shape.k_at + g * N + n0 + n, shape.silu) * (c[j] * behind[j]) : 0.0f;
             }
         }
         for (int e0 = 0; e0 < P; e0 += 64) {
@@ -357,18 +397,26 @@ __device__ __forceinline__ void load_transposed(float* to, const float* __restri
         // eight tokens by four 16-byte pieces a warp: whole sectors of every row, and two-way bank conflicts at most
         const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
         const int pieces = n_pad >> 2;
-        constexpr int ROWS = CH / 8;
+        constexpr int ROWS = CH / 8, AHEAD = 4, WARPS = LS_THREADS / 32;
         const int rounds = ROWS * ((pieces + 3) >> 2);
-        for (int r = warp; r < rounds; r += LS_THREADS / 32) {
-            const int i = (r % ROWS) * 8 + (lane & 7), piece = (r / ROWS) * 4 + (lane >> 3);
-            if (piece >= pieces) continue;
-            float4 x = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-            if (i < L && piece * 4 < N) {
-                x = *(const float4*)(from + (size_t)i * row_stride + piece * 4);
-                if (silu) x = make_float4(ls_silu(x.x), ls_silu(x.y), ls_silu(x.z), ls_silu(x.w));
+        for (int r0 = warp; r0 < rounds; r0 += AHEAD * WARPS) {        // (several loads on their way before the first store)
+            float4 x[AHEAD];
+#pragma unroll
+            for (int u = 0; u < AHEAD; ++u) {
+                const int r = r0 + u * WARPS;
+                const int i = (r % ROWS) * 8 + (lane & 7), piece = (r / ROWS) * 4 + (lane >> 3);
+                x[u] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+                if (r < rounds && i < L && piece * 4 < N) x[u] = *(const float4*)(from + (size_t)i * row_stride + piece * 4);
             }
-            float* at = to + piece * 4 * LD + i;
-            at[0] = x.x; at[LD] = x.y; at[2 * LD] = x.z; at[3 * LD] = x.w;
+#pragma unroll
+            for (int u = 0; u < AHEAD; ++u) {
+                const int r = r0 + u * WARPS;
+                const int i = (r % ROWS) * 8 + (lane & 7), piece = (r / ROWS) * 4 + (lane >> 3);
+                if (r >= rounds || piece >= pieces) continue;
+                if (silu) x[u] = make_float4(ls_silu(x[u].x), ls_silu(x[u].y), ls_silu(x[u].z), ls_silu(x[u].w));
+                float* at = to + piece * 4 * LD + i;
+                at[0] = x[u].x; at[LD] = x[u].y; at[2 * LD] = x[u].z; at[3 * LD] = x[u].w;
+            }
         }
         return;
     }
@@ -394,6 +442,9 @@ linear_state_output_kernel(const float* __restrict__ rows, const float* __restri
     float* vs = wT + CH * LD;                             // [CH][64]
     float* l = vs + CH * 64;                              // [CH]
     float* c = l + CH;                                    // [CH]
+    float* up_to = c + CH;                                // [CH]
+    float* behind = up_to + CH;                           // [CH]
+    float* spans = behind + CH;                           // [16]: the sum of l over a thread's tokens, for every row of threads
     pdl_launch_dependents();
     pdl_wait();
     const int chunk = blockIdx.x, head = blockIdx.y, s = blockIdx.z, g = head / (H / shape.groups);
@@ -402,12 +453,21 @@ linear_state_output_kernel(const float* __restrict__ rows, const float* __restri
     const bool vec_qk = ((shape.row_stride | shape.q_at | shape.k_at | N) & 3) == 0;
     const bool vec_v = ((shape.row_stride | shape.v_at | P) & 3) == 0;
     const float* base = rows + (size_t)first * shape.row_stride;
-    chunk_exponents<CH>(l, c, decay, H, head, first, L);
+    if (threadIdx.x < 32) {
+        chunk_exponents<CH>(l, c, up_to, behind, decay, H, head, first, L);
+        __syncwarp();
+        if (threadIdx.x < 16) {
+            float sum = 0.0f;
+#pragma unroll
+            for (int x = 0; x < RI; ++x) sum += l[threadIdx.x * RI + x];
+            spans[threadIdx.x] = sum;
+        }
+    }
     load_transposed<CH, LD>(qT, base + shape.q_at + g * N, shape.row_stride, N, n_pad, L, shape.silu, vec_qk);
     load_transposed<CH, LD>(kT, base + shape.k_at + g * N, shape.row_stride, N, n_pad, L, shape.silu, vec_qk);
     __syncthreads();
     const bool constant = decay.decay != nullptr;
-    const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+    const int tx = tile_x(), ty = tile_y();
     const int i0 = ty * RI, j0 = tx * RI;
     {
         float acc[RI][RI];
@@ -435,8 +495,10 @@ linear_state_output_kernel(const float* __restrict__ rows, const float* __restri
         }
         // the exponents between: what lies between the two tiles, then the tokens inside either
         float between = 0.0f;
-        if (!constant && j0 < i0)
-            for (int i = j0 + RI; i <= i0; ++i) between += l[i];
+        if (!constant && j0 < i0) {
+            for (int x = tx + 1; x < ty; ++x) between += spans[x];
+            between += l[i0];
+        }
 #pragma unroll
         for (int b = 0; b < RI; ++b) {
             const int j = j0 + b;
@@ -469,14 +531,15 @@ linear_state_output_kernel(const float* __restrict__ rows, const float* __restri
     }
     float carry[RI];
 #pragma unroll
-    for (int a = 0; a < RI; ++a) carry[a] = i0 + a < L ? span_decay(l, 0, i0 + a, constant) : 0.0f;
+    for (int a = 0; a < RI; ++a) carry[a] = i0 + a < L ? up_to[i0 + a] : 0.0f;
     const float skip = decay.skip ? decay.skip[head] : 0.0f;
     const float* before = sums + (((size_t)s * max_chunks + chunk) * H + head) * (size_t)N * P;
     float* st = kT;
-    const int j_end = min(L, (i0 / RI | 1) * RI + RI);    // (the two rows of threads of a warp walk the same keys)
+    const int j_end = min(L, ((ty | 3) + 1) * RI);        // (the four rows of threads of a warp walk the same keys)
     for (int e0 = 0; e0 < P; e0 += 64) {
         __syncthreads();                                  // the scores are in place; the tiles before have been read
         if (vec_v) {
+#pragma unroll
             for (int idx = threadIdx.x; idx < CH * 16; idx += LS_THREADS) {
                 const int j = idx >> 4, e = (idx & 15) * 4;
                 float4 x = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
@@ -486,6 +549,7 @@ linear_state_output_kernel(const float* __restrict__ rows, const float* __restri
                 }
                 *(float4*)(vs + j * 64 + e) = x;
             }
+#pragma unroll 8
             for (int idx = threadIdx.x; idx < N * 16; idx += LS_THREADS) {
                 const int n = idx >> 4, e = (idx & 15) * 4;
                 *(float4*)(st + n * 64 + e) = e0 + e < P ? *(const float4*)(before + (size_t)n * P + e0 + e) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
@@ -585,6 +649,26 @@ conv_silu_kernel(const float* __restrict__ rows, int row_stride, const float* __
     float w[CONV_HELD], u[CONV_HELD];                     // w[b], u[b]: the weight and the input of the token b back
 #pragma unroll
     for (int b = 0; b < CONV_HELD; ++b) { w[b] = held && b < taps ? weights[taps - 1 - b] : 0.0f; u[b] = 0.0f; }
+    if (held && token_seq[t0] == token_seq[t1 - 1]) {
+        // all tokens of one sequence: every input is fetched before the first is used
+        const int s = token_seq[t0], p = positions[t0], first = cu_q[s];
+        const float* ring = state + (size_t)slot_ids[s] * state_stride + ring_offset;
+        float x[CONV_TOKENS];
+#pragma unroll
+        for (int i = 0; i < CONV_TOKENS; ++i) x[i] = t0 + i < t1 ? rows[(size_t)(t0 + i) * row_stride + c] : 0.0f;
+#pragma unroll
+        for (int b = 1; b < CONV_HELD; ++b)               // u[b]: the input b tokens before this block's first
+            if (b < taps && p - b >= 0)
+                u[b] = t0 - b >= first ? rows[(size_t)(t0 - b) * row_stride + c] : ring[(size_t)((p - b) % taps) * channels + c];
+#pragma unroll
+        for (int i = 0; i < CONV_TOKENS; ++i) {
+            float sum = bias;
+#pragma unroll
+            for (int b = CONV_HELD - 1; b >= 0; --b) sum = fmaf(w[b], i >= b ? x[i >= b ? i - b : 0] : u[i < b ? b - i : 0], sum);
+            if (t0 + i < t1) out[(size_t)(t0 + i) * channels + c] = ls_silu(sum);
+        }
+        return;
+    }
     int seq = -1;
     for (int t = t0; t < t1; ++t) {
         const int s = token_seq[t], p = positions[t];
@@ -702,6 +786,55 @@ gated_norm_kernel(const float* __restrict__ y, const float* __restrict__ gate, i
         for (int i = width + threadIdx.x; i < out_stride; i += 256) out[(size_t)t * out_stride + i] = from_float<T>(0.0f);
 }
 
+// The same with a warp per (token, part) for parts of at most 128 HELD numbers (a multiple of 4) in steps of many tokens.
+template <typename T, int HELD>
+__global__ void __launch_bounds__(256)
+gated_norm_parts_kernel(const float* __restrict__ y, const float* __restrict__ gate, int gate_stride,
+                        const float* __restrict__ weight, int width, int groups, float eps, int gate_first,
+                        T* __restrict__ out, int out_stride, int items) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int item = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (item >= items) return;
+    const int t = item / groups, part = item - t * groups, size = width / groups, at = part * size;
+    const float* row = y + (size_t)t * width + at;
+    const float* g = gate + (size_t)t * gate_stride + at;
+    const float* w = weight + at;
+    T* to = out + (size_t)t * out_stride + at;
+    float4 v[HELD], z[HELD];
+#pragma unroll
+    for (int j = 0; j < HELD; ++j) {
+        const int i = 4 * (lane + 32 * j);
+        v[j] = z[j] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (i < size) { v[j] = *(const float4*)(row + i); z[j] = *(const float4*)(g + i); }
+    }
+    float squares = 0.0f;
+#pragma unroll
+    for (int j = 0; j < HELD; ++j) {
+        if (gate_first) { v[j].x *= ls_silu(z[j].x); v[j].y *= ls_silu(z[j].y); v[j].z *= ls_silu(z[j].z); v[j].w *= ls_silu(z[j].w); }
+        squares += v[j].x * v[j].x + v[j].y * v[j].y + v[j].z * v[j].z + v[j].w * v[j].w;
+    }
+    const float factor = 1.0f / sqrtf(warp_sum(squares) / (float)size + eps);
+#pragma unroll
+    for (int j = 0; j < HELD; ++j) {
+        const int i = 4 * (lane + 32 * j);
+        if (i >= size) continue;
+        const float4 x = *(const float4*)(w + i);
+        float4 r = make_float4(v[j].x * factor * x.x, v[j].y * factor * x.y, v[j].z * factor * x.z, v[j].w * factor * x.w);
+        if (!gate_first) {
+            r.x /= 1.0f + expf(-z[j].x); r.y /= 1.0f + expf(-z[j].y); r.z /= 1.0f + expf(-z[j].z); r.w /= 1.0f + expf(-z[j].w);
+        }
+        if (sizeof(T) == 4) {
+            *(float4*)(to + i) = r;
+        } else {
+            const __nv_bfloat162 lo = __floats2bfloat162_rn(r.x, r.y), hi = __floats2bfloat162_rn(r.z, r.w);
+            *(uint2*)(to + i) = make_uint2(*(const uint32_t*)&lo, *(const uint32_t*)&hi);
+        }
+    }
+    if (part == groups - 1)
+        for (int i = width + lane; i < out_stride; i += 32) out[(size_t)t * out_stride + i] = from_float<T>(0.0f);
+}
+
 static int ls_reserve(const void* kernel, size_t bytes, const char* name) {
     if (bytes <= 48 * 1024) return 0;
     if (bytes > 220 * 1024) return fail(name, "the sizes are too large for this kernel's shared memory");
@@ -712,7 +845,7 @@ static int ls_reserve(const void* kernel, size_t bytes, const char* name) {
 
 static size_t ls_output_smem(int ch, int dim) {
     const int n_pad = (dim + 3) & ~3, ld = ch + 4;
-    return (size_t)(n_pad * ld + n_pad * (ld > 64 ? ld : 64) + ch * ld + ch * 64 + 2 * ch) * sizeof(float);
+    return (size_t)(n_pad * ld + n_pad * (ld > 64 ? ld : 64) + ch * ld + ch * 64 + 4 * ch + 16) * sizeof(float);
 }
 
 // The longest chunk whose tiles fit: 64 tokens, 32, or 16.
@@ -780,7 +913,7 @@ SKV_EXPORT int skv_linear_state(const float* rows, int row_stride, int q_at, int
     const bool wide = dim > 64;
     const dim3 grid(max_chunks, heads, n_seqs);
     {
-        const size_t smem = (size_t)(ch * (wide ? 128 : 64) + ch * 64 + 3 * ch) * sizeof(float);
+        const size_t smem = (size_t)(ch * (wide ? 128 : 64) + ch * 64 + 4 * ch) * sizeof(float);
         auto kernel = ch == 64 ? (wide ? linear_state_sum_kernel<64, 8> : linear_state_sum_kernel<64, 4>)
                      : ch == 32 ? (wide ? linear_state_sum_kernel<32, 8> : linear_state_sum_kernel<32, 4>)
                                 : (wide ? linear_state_sum_kernel<16, 8> : linear_state_sum_kernel<16, 4>);
@@ -862,7 +995,12 @@ SKV_EXPORT int skv_gated_norm(const float* y, const float* gate, int gate_stride
     if (n <= 0) return 0;
     if (!y || !gate || !weight || !out || width <= 0 || groups <= 0 || width % groups || gate_stride < width || out_stride < width || groups > 65535)
         return fail("skv_gated_norm", "sizes do not agree");
-    const size_t smem = (size_t)(width / groups) * sizeof(float);
+    const int size = width / groups;
+    if ((long long)n * groups >= 2048 && (long long)n * groups <= 0x7fffffff && size <= 512 &&
+        ((size | width | gate_stride | out_stride) & 3) == 0 && (((uintptr_t)y | (uintptr_t)gate | (uintptr_t)weight | (uintptr_t)out) & 15) == 0)
+        return launch_pdl("skv_gated_norm", size <= 256 ? gated_norm_parts_kernel<skv_t, 2> : gated_norm_parts_kernel<skv_t, 4>, dim3((n * groups + 7) / 8), dim3(256), 0, stream, y, gate,
+                          gate_stride, weight, width, groups, eps, gate_first, (skv_t*)out, out_stride, n * groups);
+    const size_t smem = (size_t)size * sizeof(float);
     auto kernel = gated_norm_kernel<skv_t>;
     if (int code = ls_reserve((const void*)kernel, smem, "skv_gated_norm")) return code;
     return launch_pdl("skv_gated_norm", kernel, dim3(n, groups), dim3(256), smem, stream, y, gate, gate_stride, weight, width,

@@ -19,8 +19,43 @@ constexpr int ROUTE_THREADS = 256;
 constexpr int ROUTE_MAX_EXPERTS = 1024;
 constexpr int ROUTE_MAX_TOP = 16;
 
+// The dot product of a weight row and a float row in shared memory, a warp's share of it: VEC, sixteen bytes of the weight
+// at a time (rows of whole 16 bytes).
+template <bool VEC>
+__device__ __forceinline__ float route_dot(const float* __restrict__ w_row, const float* row, int hidden, int lane) {
+    float acc = 0.0f;
+    if (VEC) {
+        for (int w = 4 * lane; w < hidden; w += 128) {
+            const float4 a = *(const float4*)(w_row + w), b = *(const float4*)(row + w);
+            acc = fmaf(a.x, b.x, acc); acc = fmaf(a.y, b.y, acc); acc = fmaf(a.z, b.z, acc); acc = fmaf(a.w, b.w, acc);
+        }
+    } else {
+        for (int w = lane; w < hidden; w += 32) acc = fmaf(w_row[w], row[w], acc);
+    }
+    return acc;
+}
+
+template <bool VEC>
+__device__ __forceinline__ float route_dot(const __nv_bfloat16* __restrict__ w_row, const float* row, int hidden, int lane) {
+    float acc = 0.0f;
+    if (VEC) {
+        for (int w = 8 * lane; w < hidden; w += 256) {
+            const uint4 raw = *(const uint4*)(w_row + w);
+            const __nv_bfloat162* pairs = (const __nv_bfloat162*)&raw;
+            const float4 lo = *(const float4*)(row + w), hi = *(const float4*)(row + w + 4);
+            const float2 a = __bfloat1622float2(pairs[0]), b = __bfloat1622float2(pairs[1]);
+            const float2 c = __bfloat1622float2(pairs[2]), d = __bfloat1622float2(pairs[3]);
+            acc = fmaf(a.x, lo.x, acc); acc = fmaf(a.y, lo.y, acc); acc = fmaf(b.x, lo.z, acc); acc = fmaf(b.y, lo.w, acc);
+            acc = fmaf(c.x, hi.x, acc); acc = fmaf(c.y, hi.y, acc); acc = fmaf(d.x, hi.z, acc); acc = fmaf(d.y, hi.w, acc);
+        }
+    } else {
+        for (int w = lane; w < hidden; w += 32) acc = fmaf(__bfloat162float(w_row[w]), row[w], acc);
+    }
+    return acc;
+}
+
 // ---- router ------------------------------------------------------------------------------------------------------
-template <typename T>
+template <typename T, bool VEC>
 __global__ void __launch_bounds__(ROUTE_THREADS)
 route_tokens_kernel(const T* __restrict__ h, const T* __restrict__ router, const float* __restrict__ correction,
                     const T* __restrict__ shared_gate, int hidden, int experts, int top, float scale, int renormalize,
@@ -39,9 +74,7 @@ route_tokens_kernel(const T* __restrict__ h, const T* __restrict__ router, const
     const int dots = experts + (shared_gate ? 1 : 0);
     for (int e = warp; e < dots; e += ROUTE_THREADS / 32) {
         const T* w_row = e < experts ? router + (size_t)e * hidden : shared_gate;
-        float acc = 0.0f;
-        for (int w = lane; w < hidden; w += 32) acc = fmaf(to_float(w_row[w]), row[w], acc);
-        acc = warp_sum(acc);
+        const float acc = warp_sum(route_dot<VEC>(w_row, row, hidden, lane));
         if (lane == 0) {
             const float s = softmax && e < experts ? acc : 1.0f / (1.0f + expf(-acc));
             if (e < experts) {
@@ -364,6 +397,8 @@ scatter_rows_kernel(const T* __restrict__ a, const int* __restrict__ place, cons
 }
 
 // ---- the weighted sum ----------------------------------------------------------------------------------------------
+// grid (tokens, column blocks); VEC: hidden is a multiple of 4 and every pointer is 16-byte aligned.
+template <bool VEC>
 __global__ void __launch_bounds__(256)
 combine_experts_kernel(const float* __restrict__ results, const int* __restrict__ place, const float* __restrict__ weights,
                        const float* __restrict__ shared, const float* __restrict__ share, float* __restrict__ x,
@@ -379,7 +414,30 @@ combine_experts_kernel(const float* __restrict__ results, const int* __restrict_
     }
     __syncthreads();
     const float gate = shared ? (share ? share[t] : 1.0f) : 0.0f;
-    for (int w = threadIdx.x; w < hidden; w += 256) {
+    const int first = blockIdx.y * 256 + threadIdx.x, step = gridDim.y * 256;
+    if (VEC) {
+        for (int w = 4 * first; w < hidden; w += 4 * step) {
+            const size_t at = (size_t)t * hidden + w;
+            float4 total = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            for (int k = 0; k < top; ++k) {
+                const float4 r = *(const float4*)(results + (size_t)where[k] * hidden + w);
+                total.x = fmaf(weight[k], r.x, total.x); total.y = fmaf(weight[k], r.y, total.y);
+                total.z = fmaf(weight[k], r.z, total.z); total.w = fmaf(weight[k], r.w, total.w);
+            }
+            if (shared) {
+                const float4 r = *(const float4*)(shared + at);
+                total.x = fmaf(gate, r.x, total.x); total.y = fmaf(gate, r.y, total.y);
+                total.z = fmaf(gate, r.z, total.z); total.w = fmaf(gate, r.w, total.w);
+            }
+            if (add) {
+                const float4 r = *(const float4*)(x + at);
+                total = make_float4(r.x + total.x, r.y + total.y, r.z + total.z, r.w + total.w);
+            }
+            *(float4*)(x + at) = total;
+        }
+        return;
+    }
+    for (int w = first; w < hidden; w += step) {
         float total = 0.0f;
         for (int k = 0; k < top; ++k) total = fmaf(weight[k], results[(size_t)where[k] * hidden + w], total);
         if (shared) total = fmaf(gate, shared[(size_t)t * hidden + w], total);
@@ -412,7 +470,8 @@ SKV_EXPORT int skv_route_tokens(const void* h, const void* router, const float* 
     if (groups > 1 && (experts % groups != 0 || keep <= 0 || keep > groups || keep * (experts / groups) < top))
         return fail("skv_route_tokens", "groups must divide the experts, and the kept groups must hold the choices");
     const size_t smem = (size_t)(hidden + 2 * experts) * sizeof(float);
-    auto kernel = route_tokens_kernel<skv_t>;
+    const bool vec = (hidden * sizeof(skv_t)) % 16 == 0 && (((uintptr_t)router | (uintptr_t)shared_gate) & 15) == 0;
+    auto kernel = vec ? route_tokens_kernel<skv_t, true> : route_tokens_kernel<skv_t, false>;
     if (smem > 48 * 1024) {
         if (smem > 200 * 1024) return fail("skv_route_tokens", "the hidden size is too large");
         if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
@@ -500,6 +559,10 @@ SKV_EXPORT int skv_combine_experts(const float* results, const int* place, const
     if (hidden <= 0 || top <= 0 || top > ROUTE_MAX_TOP) return fail("skv_combine_experts", "1 to 16 choices a token are served");
     if (!results || !place || !x || (share && !shared))
         return fail("skv_combine_experts", "results, places, weights and the stream are needed");
-    return launch_pdl("skv_combine_experts", combine_experts_kernel, dim3(n), dim3(256), 0, stream, results, place,
+    const bool vec = hidden % 4 == 0 && (((uintptr_t)results | (uintptr_t)shared | (uintptr_t)x) & 15) == 0;
+    // a row of a step of few tokens is cut into blocks of columns that run side by side
+    const int blocks = (hidden + (vec ? 1023 : 255)) / (vec ? 1024 : 256), room = (2 * sm_count() + n - 1) / n;
+    auto kernel = vec ? combine_experts_kernel<true> : combine_experts_kernel<false>;
+    return launch_pdl("skv_combine_experts", kernel, dim3(n, blocks < room ? blocks : room), dim3(256), 0, stream, results, place,
                       weights, shared, share, x, hidden, top, add);
 }

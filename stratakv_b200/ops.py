@@ -1192,7 +1192,8 @@ class Kernels:
         ``vdim`` from ``v_at`` (``silu``: passed through silu as they are read).  The decay d is ``decay[head]`` or
         ``exp(log_decay[token, head])``, the factor c ``key_scale[token, head]`` or 1.  ``out`` ``[tokens, heads * vdim]``.
         ``state``: float32 ``[slots, floats]``, S twice from ``state_offset`` on (in the half of the last written position's
-        parity).  ``scratch``: ``linear_state_scratch`` floats."""
+        parity); steps that follow one another bring their metadata to the device with a copy on the same stream, as the
+        engine's do (a one-token step reads metadata and state before the kernel in front of it has finished).  ``scratch``: ``linear_state_scratch`` floats."""
         for name, tensor, shape in (("decay", decay, (heads,)), ("skip", skip, (heads,)),
                                     ("log_decay", log_decay, (rows.shape[0], heads)), ("key_scale", key_scale, (rows.shape[0], heads))):
             if tensor is not None:

@@ -406,11 +406,11 @@ def test_step_sizes_far_from_zero():
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("width,groups", [(48, 3), (60, 1), (126, 2), (4096, 2), (63, 7)])
-def test_gated_norms(dtype, width, groups):
+@pytest.mark.parametrize("n,width,groups", [(5, 48, 3), (5, 60, 1), (5, 126, 2), (5, 4096, 2), (5, 63, 7), (900, 48, 3), (1030, 1016, 2)])
+def test_gated_norms(dtype, n, width, groups):
     ops = kernels(dtype)
     g = torch.Generator().manual_seed(width)
-    n, padded = 5, -(-width // 8) * 8
+    padded = -(-width // 8) * 8
     y, rows, weight = torch.randn(n, width, generator=g) * 3, torch.randn(n, width + 12, generator=g), torch.rand(width, generator=g) + 0.5
     gate = rows[:, 4:4 + width].double()
     view = rows.cuda()
