@@ -362,6 +362,34 @@ __global__ void add_scaled_kernel(float* __restrict__ out, const float* __restri
         out[i] = fmaf(factor, in[i], out[i]);
 }
 
+// out[r][c] += factor * (in[r][c] + bias[c]); in may be null.  QUAD: four neighbouring numbers a thread.
+template <int QUAD>
+__global__ void add_biased_kernel(float* __restrict__ out, const float* __restrict__ in, const float* __restrict__ bias,
+                                  float factor, size_t items, int width) {
+    pdl_launch_dependents();
+    pdl_wait();
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < items; i += (size_t)gridDim.x * blockDim.x) {
+        const int c = (int)(i % (size_t)(width / QUAD)) * QUAD;
+        if (QUAD == 4) {
+            const float4 b = *(const float4*)(bias + c), x = in ? ((const float4*)in)[i] : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            float4 y = ((float4*)out)[i];
+            y.x = fmaf(factor, x.x + b.x, y.x); y.y = fmaf(factor, x.y + b.y, y.y);
+            y.z = fmaf(factor, x.z + b.z, y.z); y.w = fmaf(factor, x.w + b.w, y.w);
+            ((float4*)out)[i] = y;
+        } else {
+            out[i] = fmaf(factor, (in ? in[i] : 0.0f) + bias[c], out[i]);
+        }
+    }
+}
+
+// x[i] = cap tanh(x[i] / cap)  (a head that caps its logits)
+__global__ void softcap_inplace_kernel(float* __restrict__ x, float cap, size_t n) {
+    pdl_launch_dependents();
+    pdl_wait();
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x)
+        x[i] = cap * tanhf(x[i] / cap);
+}
+
 // x[i] *= factor  (a head that scales its logits)
 __global__ void scale_inplace_kernel(float* __restrict__ x, float factor, size_t n) {
     pdl_launch_dependents();
@@ -511,6 +539,26 @@ SKV_EXPORT int skv_add_scaled(float* out, const float* in, float factor, long lo
     if (blocks > sm_count() * 16) blocks = sm_count() * 16;
     return launch_pdl("skv_add_scaled", add_scaled_kernel, dim3((unsigned)blocks), dim3(256), 0, stream, out, in, factor,
                       (size_t)n);
+}
+
+// out float [rows, width], in the same or null, bias float [width].
+SKV_EXPORT int skv_add_biased(float* out, const float* in, const float* bias, float factor, int rows, int width, cudaStream_t stream) {
+    if (rows <= 0) return 0;
+    if (!out || !bias || width <= 0) return fail("skv_add_biased", "rows and a bias are needed");
+    const bool quad = width % 4 == 0 && (((uintptr_t)out | (uintptr_t)in | (uintptr_t)bias) & 15) == 0;
+    const size_t items = (size_t)rows * width / (quad ? 4 : 1);
+    long long blocks = ((long long)items + 255) / 256;
+    if (blocks > sm_count() * 16) blocks = sm_count() * 16;
+    return launch_pdl("skv_add_biased", quad ? add_biased_kernel<4> : add_biased_kernel<1>, dim3((unsigned)blocks), dim3(256), 0,
+                      stream, out, in, bias, factor, items, width);
+}
+
+SKV_EXPORT int skv_softcap_inplace(float* x, float cap, long long n, cudaStream_t stream) {
+    if (n <= 0) return 0;
+    if (!x || !(cap > 0.0f)) return fail("skv_softcap_inplace", "numbers and a positive cap are needed");
+    long long blocks = (n + 255) / 256;
+    if (blocks > sm_count() * 16) blocks = sm_count() * 16;
+    return launch_pdl("skv_softcap_inplace", softcap_inplace_kernel, dim3((unsigned)blocks), dim3(256), 0, stream, x, cap, (size_t)n);
 }
 
 SKV_EXPORT int skv_add_inplace(float* out, const float* in, long long n, cudaStream_t stream) {

@@ -5,12 +5,16 @@
 // value head h uses query and key head h / (heads / groups).  Per head and position p of a sequence
 //
 //   S_p = exp(l_p) S_(p-1) + c_p k_p v_p^T      (dim x vdim, zero before the first token)
-//   o_p = S_p^T q_p + skip v_p
+//   o_p = out_scale S_p^T q_p + skip v_p
 //
 // with l_p <= 0 the logarithm of the decay (one number per head, or one per token and head), c_p a factor on the key
 // (or 1) and skip a number per head (or 0).  Queries, keys and values may pass silu as they are read.
 //
-// Everything here is float.  Per sequence the cache keeps S twice, one row per slot [2][heads][dim][vdim]: a step reads
+// With a floor on the denominator (memories with exponential gates) n_p = exp(l_p) n_(p-1) + c_p k_p is kept beside S and
+// o_p = out_scale S_p^T q_p / (max(|out_scale n_p . q_p|, floor_p) + floor_eps).
+//
+// Everything here is float.  Per sequence the cache keeps S twice, one row per slot [2][heads][dim][vdim] (with a floor a
+// half is [heads][dim][vdim] and then n, [heads][dim]): a step reads
 // the half of the position before its first (by that position's parity) and writes the half of its last, so a one-token
 // step that runs twice (a graph's capture after its warm-up) computes the same thing both times.
 //
@@ -39,7 +43,15 @@ struct LinearStateDecay {
     const float* log_decay;                // [tokens][heads]: one logarithm per token and head (decay null)
     const float* key_scale;                // [tokens][heads] or null
     const float* skip;                     // [heads] or null
+    float out_scale;
+    const float* floor;                    // [tokens][heads] or null: the outputs are divided (see above)
+    float floor_eps;
 };
+
+// Floats of one half of the state, and of one chunk's sums: S of all heads, and with a floor n of all heads.
+__device__ __forceinline__ size_t ls_half(const LinearStateShape& shape, const LinearStateDecay& decay) {
+    return (size_t)shape.heads * shape.dim * (shape.vdim + (decay.floor ? 1 : 0));
+}
 
 struct LinearStateBatch {
     const int* positions;                  // [tokens]
@@ -185,9 +197,9 @@ linear_state_step_kernel(const float* __restrict__ rows, float* __restrict__ out
         for (int i = threadIdx.x; i < lanes * VEC; i += LS_THREADS) {
             const int e = cb * VEC + i;
             if (e >= P) continue;
-            float o = head_numbers[1] * v[e];
+            float o = 0.0f;
             for (int r = 0; r < per_pass; ++r) o += partial[r * lanes * VEC + i];
-            out[((size_t)t * H + head) * P + e] = o;
+            out[((size_t)t * H + head) * P + e] = fmaf(head_numbers[1], v[e], o * decay.out_scale);
         }
     }
 }
@@ -270,7 +282,8 @@ linear_state_sum_kernel(const float* __restrict__ rows, float* __restrict__ sums
     __syncthreads();
     const size_t place = ((size_t)s * max_chunks + chunk) * H + head;
     if (threadIdx.x == 0) factors[place] = up_to[L - 1];
-    float* mine = sums + place * (size_t)N * P;
+    float* chunk_sums = sums + ((size_t)s * max_chunks + chunk) * ls_half(shape, decay);
+    float* mine = chunk_sums + (size_t)head * N * P;
     const int tx = tile_x(), ty = tile_y();
     const bool vec = ((shape.row_stride | shape.k_at | shape.v_at | N | P) & 3) == 0;
     for (int n0 = 0; n0 < N; n0 += TN) {
@@ -312,6 +325,14 @@ linear_state_sum_kernel(const float* __restrict__ rows, float* __restrict__ sums
                 }
             }
             __syncthreads();
+            if (decay.floor && e0 == 0) {                 // the keys' own sum
+                float* key_sums = chunk_sums + (size_t)H * N * P + (size_t)head * N;
+                for (int n = threadIdx.x; n < TN && n0 + n < N; n += LS_THREADS) {
+                    float sum = 0.0f;
+                    for (int j = 0; j < L; ++j) sum += ks[j * TN + n];
+                    key_sums[n0 + n] = sum;
+                }
+            }
             float acc[RN][4];
 #pragma unroll
             for (int i = 0; i < RN; ++i)
@@ -355,17 +376,18 @@ linear_state_sum_kernel(const float* __restrict__ rows, float* __restrict__ sums
 // the same array would make each load wait for the one before).
 __global__ void __launch_bounds__(LS_THREADS)
 linear_state_carry_kernel(float* __restrict__ sums, const float* __restrict__ factors, int max_chunks, int chunk_len,
-                          const LinearStateShape shape, const LinearStateBatch batch) {
+                          const LinearStateShape shape, const LinearStateDecay decay, const LinearStateBatch batch) {
     pdl_launch_dependents();
     pdl_wait();
     const int H = shape.heads, cells = shape.dim * shape.vdim;
     const int head = blockIdx.y, s = blockIdx.z;
     const int at = blockIdx.x * LS_THREADS + threadIdx.x;
-    if (at >= cells) return;
+    if (at >= cells + (decay.floor ? shape.dim : 0)) return;
     const int first = batch.cu_q[s], count = batch.cu_q[s + 1] - first;
     if (count <= 0) return;
     const int p_first = batch.positions[first], p_last = p_first + count - 1;
-    const size_t half_size = (size_t)H * cells, mine = (size_t)head * cells + at;
+    const size_t half_size = ls_half(shape, decay);
+    const size_t mine = at < cells ? (size_t)head * cells + at : (size_t)H * cells + (size_t)head * shape.dim + (at - cells);
     float* slot = batch.state + (size_t)batch.slot_ids[s] * batch.state_stride + batch.state_offset;
     float S = p_first > 0 ? slot[(size_t)((p_first - 1) & 1) * half_size + mine] : 0.0f;
     const int chunks = (count + chunk_len - 1) / chunk_len;
@@ -445,13 +467,14 @@ linear_state_output_kernel(const float* __restrict__ rows, const float* __restri
     float* up_to = c + CH;                                // [CH]
     float* behind = up_to + CH;                           // [CH]
     float* spans = behind + CH;                           // [16]: the sum of l over a thread's tokens, for every row of threads
+    float* factor = spans + 16;                           // [CH]: what a token's output is multiplied by
     pdl_launch_dependents();
     pdl_wait();
     const int chunk = blockIdx.x, head = blockIdx.y, s = blockIdx.z, g = head / (H / shape.groups);
     const int first = cu_q[s] + chunk * CH, L = min(CH, cu_q[s + 1] - first);
     if (L <= 0) return;
     const bool vec_qk = ((shape.row_stride | shape.q_at | shape.k_at | N) & 3) == 0;
-    const bool vec_v = ((shape.row_stride | shape.v_at | P) & 3) == 0;
+    const bool vec_v = ((shape.row_stride | shape.v_at | P) & 3) == 0 && (!decay.floor || ((H * N) & 3) == 0);
     const float* base = rows + (size_t)first * shape.row_stride;
     if (threadIdx.x < 32) {
         chunk_exponents<CH>(l, c, up_to, behind, decay, H, head, first, L);
@@ -533,7 +556,25 @@ linear_state_output_kernel(const float* __restrict__ rows, const float* __restri
 #pragma unroll
     for (int a = 0; a < RI; ++a) carry[a] = i0 + a < L ? up_to[i0 + a] : 0.0f;
     const float skip = decay.skip ? decay.skip[head] : 0.0f;
-    const float* before = sums + (((size_t)s * max_chunks + chunk) * H + head) * (size_t)N * P;
+    const float* chunk_before = sums + ((size_t)s * max_chunks + chunk) * ls_half(shape, decay);
+    const float* before = chunk_before + (size_t)head * N * P;
+    if (decay.floor) {
+        __syncthreads();                                  // (the scores are in place)
+        if (threadIdx.x < 4 * CH) {
+            const float* n_before = chunk_before + (size_t)H * N * P + (size_t)head * N;
+            const int i = threadIdx.x >> 2, part = threadIdx.x & 3;
+            float dot = 0.0f, own = 0.0f;
+            for (int n = part; n < N; n += 4) dot = fmaf(qT[n * LD + i], n_before[n], dot);
+            for (int j = part; j <= i; j += 4) own += wT[j * LD + i];
+            dot = i < L ? fmaf(dot, up_to[i], own) : 0.0f;
+            dot += __shfl_xor_sync(0xffffffffu, dot, 1);
+            dot += __shfl_xor_sync(0xffffffffu, dot, 2);
+            if (part == 0)
+                factor[i] = i < L ? decay.out_scale / (fmaxf(fabsf(dot * decay.out_scale), decay.floor[(size_t)(first + i) * H + head]) + decay.floor_eps) : 0.0f;
+        }
+    } else if (threadIdx.x < CH) {
+        factor[threadIdx.x] = decay.out_scale;
+    }
     float* st = kT;
     const int j_end = min(L, ((ty | 3) + 1) * RI);        // (the four rows of threads of a warp walk the same keys)
     for (int e0 = 0; e0 < P; e0 += 64) {
@@ -614,8 +655,9 @@ linear_state_output_kernel(const float* __restrict__ rows, const float* __restri
             const int i = i0 + a;
             if (i >= L || e >= P) continue;
             const float4 own = *(const float4*)(vs + i * 64 + tx * 4);
-            const float o[4] = {fmaf(skip, own.x, acc[a][0]), fmaf(skip, own.y, acc[a][1]), fmaf(skip, own.z, acc[a][2]),
-                                fmaf(skip, own.w, acc[a][3])};
+            const float f = factor[i];
+            const float o[4] = {fmaf(skip, own.x, acc[a][0] * f), fmaf(skip, own.y, acc[a][1] * f), fmaf(skip, own.z, acc[a][2] * f),
+                                fmaf(skip, own.w, acc[a][3] * f)};
             float* to = out + ((size_t)(first + i) * H + head) * P + e;
             if ((P & 3) == 0) {
                 *(float4*)to = make_float4(o[0], o[1], o[2], o[3]);
@@ -643,7 +685,7 @@ conv_silu_kernel(const float* __restrict__ rows, int row_stride, const float* __
     const int c = blockIdx.x * blockDim.x + threadIdx.x;
     if (c >= channels) return;
     const int t0 = blockIdx.y * CONV_TOKENS, t1 = min(n_tokens, t0 + CONV_TOKENS);
-    const float bias = conv_b[c];
+    const float bias = conv_b ? conv_b[c] : 0.0f;
     const float* weights = conv_w + (size_t)c * taps;
     const bool held = taps <= CONV_HELD;
     float w[CONV_HELD], u[CONV_HELD];                     // w[b], u[b]: the weight and the input of the token b back
@@ -719,14 +761,94 @@ step_sizes_kernel(const float* __restrict__ rows, int row_stride, int dt_at, con
     log_decay[item] = -expf(a_log[h]) * step;
 }
 
+// ---- exponential gates with a running maximum ---------------------------------------------------------------------------
+// i = cap tanh((row + b) / cap), f = log sigmoid(cap tanh((row + b) / cap)), m_t = max(f_t + m_(t-1), i_t) with m = 0 before
+// the first token; then log_decay = f_t + m_(t-1) - m_t, key_scale = exp(i_t - m_t) and floor = exp(-m_t), each
+// [tokens][heads]: what linear_state reads.  The state of a slot holds m twice, [2][heads] from m_offset on, by the parity of
+// the last position.  A block per (head, sequence); a thread takes EG_EACH neighbouring tokens.  A run of tokens turns m into
+// max(F + m, M) with F the sum of its f, and two runs behind one another make another such pair, which the block scans.
+constexpr int EG_EACH = 4;
+
+struct GateRun { float F, M; };
+__device__ __forceinline__ GateRun behind_run(GateRun a, GateRun b) { return {a.F + b.F, fmaxf(b.F + a.M, b.M)}; }
+
+__global__ void __launch_bounds__(LS_THREADS)
+exp_gates_kernel(const float* __restrict__ rows, int row_stride, int input_at, int forget_at, const float* __restrict__ input_bias,
+                 const float* __restrict__ forget_bias, float cap, float* __restrict__ log_decay, float* __restrict__ key_scale,
+                 float* __restrict__ floor, int heads, const LinearStateBatch batch) {
+    __shared__ GateRun warp_runs[LS_THREADS / 32];
+    __shared__ float carried;
+    pdl_launch_dependents();
+    pdl_wait();
+    const int head = blockIdx.x, s = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int first = batch.cu_q[s], count = batch.cu_q[s + 1] - first;
+    if (count <= 0) return;
+    const int p_first = batch.positions[first], p_last = p_first + count - 1;
+    float* maxima = batch.state + (size_t)batch.slot_ids[s] * batch.state_stride + batch.state_offset + head;      // (m_offset)
+    if (threadIdx.x == 0) carried = p_first > 0 ? maxima[(size_t)((p_first - 1) & 1) * heads] : 0.0f;
+    const float bi = input_bias[head], bf = forget_bias[head];
+    for (int t0 = 0; t0 < count; t0 += LS_THREADS * EG_EACH) {
+        float i[EG_EACH], f[EG_EACH];
+        const int mine = t0 + threadIdx.x * EG_EACH;
+        GateRun run = {0.0f, -INFINITY};
+#pragma unroll
+        for (int e = 0; e < EG_EACH; ++e) {
+            i[e] = -INFINITY;
+            f[e] = 0.0f;
+            if (mine + e < count) {
+                const float* row = rows + (size_t)(first + mine + e) * row_stride;
+                i[e] = cap * tanhf((row[input_at + head] + bi) / cap);
+                const float z = cap * tanhf((row[forget_at + head] + bf) / cap);
+                f[e] = fminf(z, 0.0f) - log1pf(expf(-fabsf(z)));
+            }
+        }
+#pragma unroll
+        for (int e = 0; e < EG_EACH; ++e) run = behind_run(run, {f[e], i[e]});
+        // the runs of the lanes below, then of the warps below
+        GateRun upto = run;
+#pragma unroll
+        for (int offset = 1; offset < 32; offset <<= 1) {
+            const GateRun below = {__shfl_up_sync(0xffffffffu, upto.F, offset), __shfl_up_sync(0xffffffffu, upto.M, offset)};
+            if (lane >= offset) upto = behind_run(below, upto);
+        }
+        if (lane == 31) warp_runs[warp] = upto;
+        GateRun before = {__shfl_up_sync(0xffffffffu, upto.F, 1), __shfl_up_sync(0xffffffffu, upto.M, 1)};
+        if (lane == 0) before = {0.0f, -INFINITY};
+        __syncthreads();
+        GateRun lower = {0.0f, -INFINITY};
+        for (int x = 0; x < warp; ++x) lower = behind_run(lower, warp_runs[x]);
+        before = behind_run(lower, before);
+        float m = fmaxf(before.F + carried, before.M);
+        __syncthreads();                                  // (everybody has read what was carried)
+#pragma unroll
+        for (int e = 0; e < EG_EACH; ++e) {
+            if (mine + e >= count) break;
+            const float top = fmaxf(f[e] + m, i[e]);
+            const size_t at = (size_t)(first + mine + e) * heads + head;
+            log_decay[at] = f[e] + m - top;
+            key_scale[at] = expf(i[e] - top);
+            floor[at] = expf(-top);
+            m = top;
+            if (mine + e == min(count, t0 + LS_THREADS * EG_EACH) - 1) {       // the last token of this round
+                carried = m;
+                if (mine + e == count - 1) maxima[(size_t)(p_last & 1) * heads] = m;
+            }
+        }
+        __syncthreads();
+    }
+}
+
 // ---- a norm with a gate ------------------------------------------------------------------------------------------------
+enum { GATE_SIGMOID = 0, GATE_SILU_FIRST = 1, GATE_SILU = 2 };
+__device__ __forceinline__ float gate_after(float z, int mode) { return (mode == GATE_SILU ? z : 1.0f) / (1.0f + expf(-z)); }
+
 // out = gated norm of float rows y [tokens, width]: the row in `groups` equal parts, each divided by its own root mean
-// square, times a weight, and a gate on every number: gate_first, silu(gate) before the norm; else sigmoid(gate) after it.
+// square, times a weight, and a gate on every number: sigmoid(gate) or silu(gate) after the norm, or silu(gate) before it.
 // A block per (token, part); the part stays in shared memory between the two passes.
 template <typename T>
 __global__ void __launch_bounds__(256)
 gated_norm_kernel(const float* __restrict__ y, const float* __restrict__ gate, int gate_stride, const float* __restrict__ weight,
-                  int width, int groups, float eps, int gate_first, T* __restrict__ out, int out_stride) {
+                  int width, int groups, float eps, int mode, T* __restrict__ out, int out_stride) {
     extern __shared__ __align__(16) float gn_part[];
     __shared__ float scratch[33];
     pdl_launch_dependents();
@@ -742,7 +864,7 @@ gated_norm_kernel(const float* __restrict__ y, const float* __restrict__ gate, i
     if (vec) {
         for (int i = 4 * threadIdx.x; i < size; i += 1024) {
             float4 v = *(const float4*)(row + i);
-            if (gate_first) {
+            if (mode == GATE_SILU_FIRST) {
                 const float4 z = *(const float4*)(g + i);
                 v.x *= ls_silu(z.x); v.y *= ls_silu(z.y); v.z *= ls_silu(z.z); v.w *= ls_silu(z.w);
             }
@@ -753,7 +875,7 @@ gated_norm_kernel(const float* __restrict__ y, const float* __restrict__ gate, i
     } else {
         for (int i = threadIdx.x; i < size; i += 256) {
             float v = row[i];
-            if (gate_first) v *= ls_silu(g[i]);
+            if (mode == GATE_SILU_FIRST) v *= ls_silu(g[i]);
             squares = fmaf(v, v, squares);
             gn_part[i] = v;
         }
@@ -764,9 +886,9 @@ gated_norm_kernel(const float* __restrict__ y, const float* __restrict__ gate, i
             float4 v = *(const float4*)(gn_part + i);
             const float4 x = *(const float4*)(w + i);
             v.x *= factor * x.x; v.y *= factor * x.y; v.z *= factor * x.z; v.w *= factor * x.w;
-            if (!gate_first) {
+            if (mode != GATE_SILU_FIRST) {
                 const float4 z = *(const float4*)(g + i);
-                v.x /= 1.0f + expf(-z.x); v.y /= 1.0f + expf(-z.y); v.z /= 1.0f + expf(-z.z); v.w /= 1.0f + expf(-z.w);
+                v.x *= gate_after(z.x, mode); v.y *= gate_after(z.y, mode); v.z *= gate_after(z.z, mode); v.w *= gate_after(z.w, mode);
             }
             if (sizeof(T) == 4) {
                 *(float4*)(to + i) = v;
@@ -778,7 +900,7 @@ gated_norm_kernel(const float* __restrict__ y, const float* __restrict__ gate, i
     } else {
         for (int i = threadIdx.x; i < size; i += 256) {
             float v = gn_part[i] * factor * w[i];
-            if (!gate_first) v /= 1.0f + expf(-g[i]);
+            if (mode != GATE_SILU_FIRST) v *= gate_after(g[i], mode);
             to[i] = from_float<T>(v);
         }
     }
@@ -790,7 +912,7 @@ gated_norm_kernel(const float* __restrict__ y, const float* __restrict__ gate, i
 template <typename T, int HELD>
 __global__ void __launch_bounds__(256)
 gated_norm_parts_kernel(const float* __restrict__ y, const float* __restrict__ gate, int gate_stride,
-                        const float* __restrict__ weight, int width, int groups, float eps, int gate_first,
+                        const float* __restrict__ weight, int width, int groups, float eps, int mode,
                         T* __restrict__ out, int out_stride, int items) {
     pdl_launch_dependents();
     pdl_wait();
@@ -811,7 +933,7 @@ gated_norm_parts_kernel(const float* __restrict__ y, const float* __restrict__ g
     float squares = 0.0f;
 #pragma unroll
     for (int j = 0; j < HELD; ++j) {
-        if (gate_first) { v[j].x *= ls_silu(z[j].x); v[j].y *= ls_silu(z[j].y); v[j].z *= ls_silu(z[j].z); v[j].w *= ls_silu(z[j].w); }
+        if (mode == GATE_SILU_FIRST) { v[j].x *= ls_silu(z[j].x); v[j].y *= ls_silu(z[j].y); v[j].z *= ls_silu(z[j].z); v[j].w *= ls_silu(z[j].w); }
         squares += v[j].x * v[j].x + v[j].y * v[j].y + v[j].z * v[j].z + v[j].w * v[j].w;
     }
     const float factor = 1.0f / sqrtf(warp_sum(squares) / (float)size + eps);
@@ -821,8 +943,8 @@ gated_norm_parts_kernel(const float* __restrict__ y, const float* __restrict__ g
         if (i >= size) continue;
         const float4 x = *(const float4*)(w + i);
         float4 r = make_float4(v[j].x * factor * x.x, v[j].y * factor * x.y, v[j].z * factor * x.z, v[j].w * factor * x.w);
-        if (!gate_first) {
-            r.x /= 1.0f + expf(-z[j].x); r.y /= 1.0f + expf(-z[j].y); r.z /= 1.0f + expf(-z[j].z); r.w /= 1.0f + expf(-z[j].w);
+        if (mode != GATE_SILU_FIRST) {
+            r.x *= gate_after(z[j].x, mode); r.y *= gate_after(z[j].y, mode); r.z *= gate_after(z[j].z, mode); r.w *= gate_after(z[j].w, mode);
         }
         if (sizeof(T) == 4) {
             *(float4*)(to + i) = r;
@@ -845,7 +967,7 @@ static int ls_reserve(const void* kernel, size_t bytes, const char* name) {
 
 static size_t ls_output_smem(int ch, int dim) {
     const int n_pad = (dim + 3) & ~3, ld = ch + 4;
-    return (size_t)(n_pad * ld + n_pad * (ld > 64 ? ld : 64) + ch * ld + ch * 64 + 4 * ch + 16) * sizeof(float);
+    return (size_t)(n_pad * ld + n_pad * (ld > 64 ? ld : 64) + ch * ld + ch * 64 + 5 * ch + 16) * sizeof(float);
 }
 
 // The longest chunk whose tiles fit: 64 tokens, 32, or 16.
@@ -853,7 +975,7 @@ static int ls_chunk(int dim) {
     return ls_output_smem(64, dim) <= 200 * 1024 ? 64 : (ls_output_smem(32, dim) <= 200 * 1024 ? 32 : 16);
 }
 
-static int ls_check(const char* name, const LinearStateShape& shape, const LinearStateBatch& batch) {
+static int ls_check(const char* name, const LinearStateShape& shape, const LinearStateBatch& batch, bool with_floor) {
     if (shape.heads <= 0 || shape.groups <= 0 || shape.heads % shape.groups || shape.dim <= 0 || shape.vdim <= 0)
         return fail(name, "heads must be a positive multiple of the query and key heads, and sizes positive");
     if (shape.heads > 65535) return fail(name, "too many heads");
@@ -863,8 +985,8 @@ static int ls_check(const char* name, const LinearStateShape& shape, const Linea
         return fail(name, "queries, keys and values must lie inside a row");
     if (!batch.positions || !batch.cu_q || !batch.slot_ids || !batch.state)
         return fail(name, "the step's metadata and the state are needed");
-    if (batch.state_offset < 0 || batch.state_offset + 2LL * shape.heads * shape.dim * shape.vdim > batch.state_stride)
-        return fail(name, "a slot's state is too small: 2 * heads * dim * vdim floats are needed");
+    if (batch.state_offset < 0 || batch.state_offset + 2LL * shape.heads * shape.dim * (shape.vdim + (with_floor ? 1 : 0)) > batch.state_stride)
+        return fail(name, "a slot's state is too small: two halves of heads * dim * vdim floats (and heads * dim with a floor) are needed");
     return 0;
 }
 
@@ -873,17 +995,17 @@ static int ls_check(const char* name, const LinearStateShape& shape, const Linea
 using namespace skv;
 
 // Floats of scratch for a step whose longest sequence brings max_q_len tokens (0 for one token a sequence).
-SKV_EXPORT long long skv_linear_state_scratch(int n_seqs, int max_q_len, int heads, int dim, int vdim) {
-    if (max_q_len <= 1) return 0;
+SKV_EXPORT long long skv_linear_state_scratch(int n_seqs, int max_q_len, int heads, int dim, int vdim, int with_floor) {
+    if (max_q_len <= 1 && !with_floor) return 0;
     const int ch = ls_chunk(dim);
-    return (long long)n_seqs * ((max_q_len + ch - 1) / ch) * heads * ((long long)dim * vdim + 1);
+    return (long long)n_seqs * ((max_q_len + ch - 1) / ch) * heads * ((long long)dim * (vdim + (with_floor ? 1 : 0)) + 1);
 }
 
 // rows: float [n_tokens, row_stride]; out: float [n_tokens, heads * vdim].  decay [heads], or log_decay [n_tokens, heads];
 // key_scale [n_tokens, heads] and skip [heads] may be null.  state: float [slots][state_stride].
 SKV_EXPORT int skv_linear_state(const float* rows, int row_stride, int q_at, int k_at, int v_at, int silu, const float* decay,
-                                const float* log_decay, const float* key_scale, const float* skip, float* out,
-                                float* scratch, int n_tokens, int n_seqs, int heads, int groups, int dim, int vdim,
+                                const float* log_decay, const float* key_scale, const float* skip, float out_scale,
+                                const float* floor, float floor_eps, float* out, float* scratch, int n_tokens, int n_seqs, int heads, int groups, int dim, int vdim,
                                 int max_q_len, const int* positions, const int* token_seq, const int* cu_q,
                                 const int* slot_ids, float* state, long long state_stride, long long state_offset,
                                 cudaStream_t stream) {
@@ -892,11 +1014,11 @@ SKV_EXPORT int skv_linear_state(const float* rows, int row_stride, int q_at, int
     if (!rows || !out || (!decay && !log_decay)) return fail(name, "rows, a decay and a place for the result are needed");
     if (n_seqs > 65535 || max_q_len <= 0) return fail(name, "too many sequences in one step, or no tokens");
     const LinearStateShape shape = {heads, groups, dim, vdim, row_stride, q_at, k_at, v_at, silu};
-    const LinearStateDecay decays = {decay, log_decay, key_scale, skip};
+    const LinearStateDecay decays = {decay, log_decay, key_scale, skip, out_scale, floor, floor_eps};
     const LinearStateBatch batch = {positions, cu_q, slot_ids, state, state_stride, state_offset};
-    if (int code = ls_check(name, shape, batch)) return code;
+    if (int code = ls_check(name, shape, batch, floor != nullptr)) return code;
     if (((uintptr_t)rows | (uintptr_t)out | (uintptr_t)state | (uintptr_t)scratch) & 15) return fail(name, "operands must be 16-byte aligned");
-    if (max_q_len == 1) {
+    if (max_q_len == 1 && !floor) {
         if (n_tokens != n_seqs) return fail(name, "one token a sequence means as many tokens as sequences");
         ConvStep none = {};
         const bool vec = vdim % 4 == 0 && state_stride % 4 == 0 && state_offset % 4 == 0;
@@ -909,7 +1031,8 @@ SKV_EXPORT int skv_linear_state(const float* rows, int row_stride, int q_at, int
     const int ch = ls_chunk(dim), max_chunks = (max_q_len + ch - 1) / ch;
     if (ls_output_smem(ch, dim) > 220 * 1024) return fail(name, "the head size is too large for this kernel's shared memory");
     float* sums = scratch;
-    float* factors = scratch + (size_t)n_seqs * max_chunks * heads * dim * vdim;
+    const int per_key = vdim + (floor ? 1 : 0);           // numbers a key channel keeps
+    float* factors = scratch + (size_t)n_seqs * max_chunks * heads * dim * per_key;
     const bool wide = dim > 64;
     const dim3 grid(max_chunks, heads, n_seqs);
     {
@@ -921,8 +1044,8 @@ SKV_EXPORT int skv_linear_state(const float* rows, int row_stride, int q_at, int
         if (int code = launch_pdl(name, kernel, grid, dim3(LS_THREADS), smem, stream, rows, sums, factors, max_chunks, shape, decays, cu_q))
             return code;
     }
-    if (int code = launch_pdl(name, linear_state_carry_kernel, dim3((dim * vdim + LS_THREADS - 1) / LS_THREADS, heads, n_seqs),
-                              dim3(LS_THREADS), 0, stream, sums, (const float*)factors, max_chunks, ch, shape, batch))
+    if (int code = launch_pdl(name, linear_state_carry_kernel, dim3((dim * per_key + LS_THREADS - 1) / LS_THREADS, heads, n_seqs),
+                              dim3(LS_THREADS), 0, stream, sums, (const float*)factors, max_chunks, ch, shape, decays, batch))
         return code;
     const size_t smem = ls_output_smem(ch, dim);
     auto kernel = ch == 64 ? linear_state_output_kernel<64> : (ch == 32 ? linear_state_output_kernel<32> : linear_state_output_kernel<16>);
@@ -946,10 +1069,10 @@ SKV_EXPORT int skv_mamba2_step(const float* rows, int row_stride, const float* c
     if (n_seqs > 65535) return fail(name, "too many sequences in one step");
     const int inner = heads * vdim, channels = inner + 2 * groups * dim;
     const LinearStateShape shape = {heads, groups, dim, vdim, row_stride, inner + groups * dim, inner, 0, 0};
-    const LinearStateDecay decays = {nullptr, nullptr, nullptr, skip};
+    const LinearStateDecay decays = {nullptr, nullptr, nullptr, skip, 1.0f, nullptr, 0.0f};
     const LinearStateBatch batch = {positions, cu_q, slot_ids, state, state_stride, state_offset};
     const ConvStep conv = {conv_w, conv_b, dt_bias, a_log, taps, channels, dt_at, ring_offset};
-    if (int code = ls_check(name, shape, batch)) return code;
+    if (int code = ls_check(name, shape, batch, false)) return code;
     if (dt_at < 0 || dt_at + heads > row_stride || ring_offset < 0 ||
         (taps > 1 && ring_offset + (long long)taps * channels > state_stride))
         return fail(name, "the step sizes must lie inside a row and the ring inside a slot's state");
@@ -968,7 +1091,7 @@ SKV_EXPORT int skv_conv_silu(const float* rows, int row_stride, const float* con
                              const int* slot_ids, const float* state, long long state_stride, long long ring_offset,
                              cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
-    if (!rows || !conv_w || !conv_b || !out || !positions || !token_seq || !cu_q || !slot_ids || (taps > 1 && !state))
+    if (!rows || !conv_w || !out || !positions || !token_seq || !cu_q || !slot_ids || (taps > 1 && !state))
         return fail("skv_conv_silu", "a pointer is missing");
     if (channels <= 0 || taps <= 0 || row_stride < channels || (taps > 1 && (ring_offset < 0 || ring_offset + (long long)taps * channels > state_stride)))
         return fail("skv_conv_silu", "sizes do not agree");
@@ -991,18 +1114,37 @@ SKV_EXPORT int skv_step_sizes(const float* rows, int row_stride, int dt_at, cons
 
 // y float [n, width], gate float rows gate_stride apart, weight float [width], out [n, out_stride] in the compute dtype.
 SKV_EXPORT int skv_gated_norm(const float* y, const float* gate, int gate_stride, const float* weight, int width, int groups,
-                              float eps, int gate_first, void* out, int out_stride, int n, cudaStream_t stream) {
+                              float eps, int mode, void* out, int out_stride, int n, cudaStream_t stream) {
     if (n <= 0) return 0;
-    if (!y || !gate || !weight || !out || width <= 0 || groups <= 0 || width % groups || gate_stride < width || out_stride < width || groups > 65535)
+    if (!y || !gate || !weight || !out || width <= 0 || groups <= 0 || width % groups || gate_stride < width || out_stride < width || groups > 65535 ||
+        mode < GATE_SIGMOID || mode > GATE_SILU)
         return fail("skv_gated_norm", "sizes do not agree");
     const int size = width / groups;
     if ((long long)n * groups >= 2048 && (long long)n * groups <= 0x7fffffff && size <= 512 &&
         ((size | width | gate_stride | out_stride) & 3) == 0 && (((uintptr_t)y | (uintptr_t)gate | (uintptr_t)weight | (uintptr_t)out) & 15) == 0)
         return launch_pdl("skv_gated_norm", size <= 256 ? gated_norm_parts_kernel<skv_t, 2> : gated_norm_parts_kernel<skv_t, 4>, dim3((n * groups + 7) / 8), dim3(256), 0, stream, y, gate,
-                          gate_stride, weight, width, groups, eps, gate_first, (skv_t*)out, out_stride, n * groups);
+                          gate_stride, weight, width, groups, eps, mode, (skv_t*)out, out_stride, n * groups);
     const size_t smem = (size_t)size * sizeof(float);
     auto kernel = gated_norm_kernel<skv_t>;
     if (int code = ls_reserve((const void*)kernel, smem, "skv_gated_norm")) return code;
     return launch_pdl("skv_gated_norm", kernel, dim3(n, groups), dim3(256), smem, stream, y, gate, gate_stride, weight, width,
-                      groups, eps, gate_first, (skv_t*)out, out_stride);
+                      groups, eps, mode, (skv_t*)out, out_stride);
+}
+
+// rows float [n_tokens, row_stride] with the gates' logits at columns input_at and forget_at; log_decay, key_scale and floor
+// float [n_tokens, heads]; a slot's state holds [2][heads] floats from m_offset on.
+SKV_EXPORT int skv_exp_gates(const float* rows, int row_stride, int input_at, int forget_at, const float* input_bias,
+                             const float* forget_bias, float cap, float* log_decay, float* key_scale, float* floor, int heads,
+                             int n_seqs, const int* positions, const int* token_seq, const int* cu_q, const int* slot_ids,
+                             float* state, long long state_stride, long long m_offset, cudaStream_t stream) {
+    const char* name = "skv_exp_gates";
+    if (n_seqs <= 0) return 0;
+    if (!rows || !input_bias || !forget_bias || !log_decay || !key_scale || !floor || !positions || !cu_q || !slot_ids || !state)
+        return fail(name, "a pointer is missing");
+    if (heads <= 0 || n_seqs > 65535 || !(cap > 0.0f) || input_at < 0 || forget_at < 0 || input_at + heads > row_stride ||
+        forget_at + heads > row_stride || m_offset < 0 || m_offset + 2LL * heads > state_stride)
+        return fail(name, "the gates must lie inside a row and the maxima inside a slot's state");
+    const LinearStateBatch batch = {positions, cu_q, slot_ids, state, state_stride, m_offset};
+    return launch_pdl(name, exp_gates_kernel, dim3(heads, n_seqs), dim3(LS_THREADS), 0, stream, rows, row_stride, input_at,
+                      forget_at, input_bias, forget_bias, cap, log_decay, key_scale, floor, heads, batch);
 }

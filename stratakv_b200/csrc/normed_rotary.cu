@@ -1,5 +1,6 @@
 // From the float rows [q | k | v] of a fused projection to attention's inputs, in one kernel with a block per token:
 //
+//   bias   added to the whole row first, if there is one;
 //   q, k   an RMS norm with a weight over all query heads together and one over all key heads together (either may be
 //          left out), then rotary positions on the first `rotated` numbers of every head (pairs (2i, 2i+1) or
 //          (i, i + rotated/2));
@@ -21,6 +22,7 @@ struct NormedRotary {
     const float* q_weight;         // [heads * dim] or null
     const float* k_weight;         // [kv_heads * dim] or null
     float eps;
+    const float* bias;             // [heads * dim + kv_heads * (dim + vdim)] or null
     const float2* cos_sin;         // [positions][rotated / 2] or null
     int rotated, interleaved;
     const float* mix;              // one number, or null
@@ -42,8 +44,9 @@ __device__ __forceinline__ float2 block_sum2(float a, float b, float* scratch) {
     return make_float2(ta, tb);
 }
 
-// VEC: head sizes, widths and the row stride are multiples of 4, the rotation is interleaved (or absent) and every pointer
-// is 16-byte aligned: four neighbouring numbers (two pairs) a thread and round.
+// VEC: head sizes, widths and the row stride are multiples of 4, the rotation is interleaved (or absent, or its halves are
+// multiples of 4) and every pointer is 16-byte aligned: four neighbouring numbers (two pairs, or one side of four) a thread
+// and round.
 template <typename T, bool VEC>
 __global__ void __launch_bounds__(NR_THREADS)
 normed_rotary_kernel(const float* __restrict__ rows, const int* __restrict__ positions, const int* __restrict__ token_seq,
@@ -57,6 +60,18 @@ normed_rotary_kernel(const float* __restrict__ rows, const int* __restrict__ pos
     const int nq = a.heads * a.dim, nk = a.kv_heads * a.dim, nv = a.kv_heads * a.vdim;
     const float* k = q + nq;
     const float* v = k + nk;
+    const float* bq = a.bias;                           // (null: no bias anywhere)
+    const float* bk = bq ? bq + nq : nullptr;
+    const float* bv = bq ? bk + nk : nullptr;
+    auto load4 = [](const float* x, const float* b, int c) {
+        float4 z = *(const float4*)(x + c);
+        if (b) {
+            const float4 w = *(const float4*)(b + c);
+            z.x += w.x; z.y += w.y; z.z += w.z; z.w += w.w;
+        }
+        return z;
+    };
+    auto load1 = [](const float* x, const float* b, int c) { return b ? x[c] + b[c] : x[c]; };
     const int pos = positions[t];
     size_t base = 0;                                    // the token's row of key head 0, in rows of one head's vector
     if (a.write_kv) base = (size_t)block_table[(size_t)token_seq[t] * table_width + pos / block_size] * a.kv_heads * block_size + pos % block_size;
@@ -67,17 +82,17 @@ normed_rotary_kernel(const float* __restrict__ rows, const int* __restrict__ pos
         if (VEC) {
             if (a.q_weight)
                 for (int i = 4 * threadIdx.x; i < nq; i += 4 * NR_THREADS) {
-                    const float4 x = *(const float4*)(q + i);
+                    const float4 x = load4(q, bq, i);
                     sq = fmaf(x.x, x.x, sq); sq = fmaf(x.y, x.y, sq); sq = fmaf(x.z, x.z, sq); sq = fmaf(x.w, x.w, sq);
                 }
             if (a.k_weight)
                 for (int i = 4 * threadIdx.x; i < nk; i += 4 * NR_THREADS) {
-                    const float4 x = *(const float4*)(k + i);
+                    const float4 x = load4(k, bk, i);
                     sk = fmaf(x.x, x.x, sk); sk = fmaf(x.y, x.y, sk); sk = fmaf(x.z, x.z, sk); sk = fmaf(x.w, x.w, sk);
                 }
         } else {
-            if (a.q_weight) for (int i = threadIdx.x; i < nq; i += NR_THREADS) sq = fmaf(q[i], q[i], sq);
-            if (a.k_weight) for (int i = threadIdx.x; i < nk; i += NR_THREADS) sk = fmaf(k[i], k[i], sk);
+            if (a.q_weight) for (int i = threadIdx.x; i < nq; i += NR_THREADS) { const float x = load1(q, bq, i); sq = fmaf(x, x, sq); }
+            if (a.k_weight) for (int i = threadIdx.x; i < nk; i += NR_THREADS) { const float x = load1(k, bk, i); sk = fmaf(x, x, sk); }
         }
         const float2 sums = block_sum2(sq, sk, scratch);
         if (a.q_weight) q_factor = 1.0f / sqrtf(sums.x / (float)nq + a.eps);
@@ -100,25 +115,40 @@ normed_rotary_kernel(const float* __restrict__ rows, const int* __restrict__ pos
             const int head = index / quads, d = (index - head * quads) * 4;
             float4 x = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
             if (d < a.dim) {
-                const int c = head * a.dim + d;
-                x = *(const float4*)((is_query ? q : k) + c);
                 const float* weight = is_query ? a.q_weight : a.k_weight;
-                if (weight) {
-                    const float4 w = *(const float4*)(weight + c);
-                    const float f = is_query ? q_factor : k_factor;
-                    x.x *= f * w.x; x.y *= f * w.y; x.z *= f * w.z; x.w *= f * w.w;
-                }
-                if (d < a.rotated) {
-                    const float2 cs = angles[d >> 1];
-                    const float u = x.x * cs.x - x.y * cs.y;
-                    x.y = x.y * cs.x + x.x * cs.y;
-                    x.x = u;
-                }
-                if (d + 2 < a.rotated) {
-                    const float2 cs = angles[(d >> 1) + 1];
-                    const float u = x.z * cs.x - x.w * cs.y;
-                    x.w = x.w * cs.x + x.z * cs.y;
-                    x.z = u;
+                const float f = is_query ? q_factor : k_factor;
+                auto normed4 = [&](int c) {
+                    float4 z = load4(is_query ? q : k, is_query ? bq : bk, c);
+                    if (weight) {
+                        const float4 w = *(const float4*)(weight + c);
+                        z.x *= f * w.x; z.y *= f * w.y; z.z *= f * w.z; z.w *= f * w.w;
+                    }
+                    return z;
+                };
+                const int c = head * a.dim + d;
+                x = normed4(c);
+                if (a.interleaved) {
+                    if (d < a.rotated) {
+                        const float2 cs = angles[d >> 1];
+                        const float u = x.x * cs.x - x.y * cs.y;
+                        x.y = x.y * cs.x + x.x * cs.y;
+                        x.x = u;
+                    }
+                    if (d + 2 < a.rotated) {
+                        const float2 cs = angles[(d >> 1) + 1];
+                        const float u = x.z * cs.x - x.w * cs.y;
+                        x.w = x.w * cs.x + x.z * cs.y;
+                        x.z = u;
+                    }
+                } else if (d < a.rotated) {
+                    const int half = a.rotated >> 1;
+                    const bool low = d < half;
+                    const float4 m = normed4(low ? c + half : c - half);
+                    const float sign = low ? -1.0f : 1.0f;
+                    const float2* turn = angles + (low ? d : d - half);
+                    const float2 t0 = turn[0], t1 = turn[1], t2 = turn[2], t3 = turn[3];
+                    x = make_float4(x.x * t0.x + sign * m.x * t0.y, x.y * t1.x + sign * m.y * t1.y,
+                                    x.z * t2.x + sign * m.z * t2.y, x.w * t3.x + sign * m.w * t3.y);
                 }
             }
             store4(is_query ? q_out + ((size_t)t * a.heads + head) * a.q_width + d
@@ -130,7 +160,7 @@ normed_rotary_kernel(const float* __restrict__ rows, const int* __restrict__ pos
             float4 x = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
             if (d < a.vdim) {
                 const size_t c = (size_t)head * a.vdim + d;
-                x = *(const float4*)(v + c);
+                x = load4(v, bv, (int)c);
                 if (a.keep) *(float4*)(a.keep + (size_t)t * nv + c) = x;
                 if (a.mix) {
                     const float4 f = *(const float4*)(a.first + (size_t)t * nv + c);
@@ -146,7 +176,7 @@ normed_rotary_kernel(const float* __restrict__ rows, const int* __restrict__ pos
     auto value_at = [&](bool is_query, int head, int d) {
         const int c = head * a.dim + d;
         const float* weight = is_query ? a.q_weight : a.k_weight;
-        const float x = (is_query ? q : k)[c];
+        const float x = load1(is_query ? q : k, is_query ? bq : bk, c);
         return weight ? x * ((is_query ? q_factor : k_factor) * weight[c]) : x;
     };
     const int q_items = a.heads * a.q_width, k_items = a.write_kv ? a.kv_heads * a.q_width : 0;
@@ -173,7 +203,7 @@ normed_rotary_kernel(const float* __restrict__ rows, const int* __restrict__ pos
         float x = 0.0f;
         if (d < a.vdim) {
             const size_t c = (size_t)head * a.vdim + d;
-            x = v[c];
+            x = load1(v, bv, (int)c);
             if (a.keep) a.keep[(size_t)t * nv + c] = x;
             if (a.mix) x = fmaf(mix, a.first[(size_t)t * nv + c], (1.0f - mix) * x);
         }
@@ -187,7 +217,7 @@ using namespace skv;
 
 // rows float [n, row_stride]: [heads * dim queries | kv_heads * dim keys | kv_heads * vdim values | ...]; q_out
 // [n, heads * q_width], k_cache [blocks, kv_heads, block_size, q_width], v_cache [.., v_width] in the compute dtype.
-SKV_EXPORT int skv_normed_rotary(const float* rows, int row_stride, const float* q_weight, const float* k_weight, float eps,
+SKV_EXPORT int skv_normed_rotary(const float* rows, int row_stride, const float* bias, const float* q_weight, const float* k_weight, float eps,
                                  const float* cos_sin, int rotated, int interleaved, const float* mix, const float* first,
                                  float* keep, const int* positions, const int* token_seq, const int* block_table,
                                  int table_width, void* q_out, void* k_cache, void* v_cache, int n, int heads, int kv_heads,
@@ -200,10 +230,10 @@ SKV_EXPORT int skv_normed_rotary(const float* rows, int row_stride, const float*
         return fail(name, "sizes do not agree");
     if (!rows || !positions || !token_seq || !block_table || !q_out || !k_cache || !v_cache || (rotated > 0 && !cos_sin) || (mix && !first))
         return fail(name, "a pointer is missing");
-    const NormedRotary a = {heads, kv_heads, dim, vdim, q_width, v_width, row_stride, q_weight, k_weight, eps,
+    const NormedRotary a = {heads, kv_heads, dim, vdim, q_width, v_width, row_stride, q_weight, k_weight, eps, bias,
                             (const float2*)(rotated > 0 ? cos_sin : nullptr), rotated, interleaved, mix, first, keep, write_kv};
-    const bool vec = ((dim | vdim | q_width | v_width | row_stride) & 3) == 0 && (interleaved || rotated == 0) &&
-                     (((uintptr_t)rows | (uintptr_t)q_weight | (uintptr_t)k_weight | (uintptr_t)first | (uintptr_t)keep |
+    const bool vec = ((dim | vdim | q_width | v_width | row_stride) & 3) == 0 && (interleaved || rotated % 8 == 0) &&
+                     (((uintptr_t)rows | (uintptr_t)bias | (uintptr_t)q_weight | (uintptr_t)k_weight | (uintptr_t)first | (uintptr_t)keep |
                        (uintptr_t)q_out | (uintptr_t)k_cache | (uintptr_t)v_cache) & 15) == 0;
     auto kernel = vec ? normed_rotary_kernel<skv_t, true> : normed_rotary_kernel<skv_t, false>;
     return launch_pdl(name, kernel, dim3(n), dim3(NR_THREADS), 0, stream, rows, positions, token_seq, block_table, table_width,

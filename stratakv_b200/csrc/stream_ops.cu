@@ -7,7 +7,7 @@
 //
 // Both can hand the next reader its input in the same pass: with next_out, the new row of the stream is normed
 // with next_gamma and next_eps and written in the compute dtype, so the norm in front of the next sublayer needs no
-// kernel of its own.  Everything is float but the tables and weights, which are read in the compute dtype.
+// kernel of its own; rmsnorm_add without next_gamma writes the new row as it is, for sublayers that read the stream itself.  Everything is float but the tables and weights, which are read in the compute dtype.
 #include "common.cuh"
 
 namespace skv {
@@ -35,8 +35,12 @@ __global__ void rmsnorm_add_kernel(const float* __restrict__ y, const float* __r
         squares = fmaf(v, v, squares);
     }
     if (!next_out) return;
-    const float next_inverse = 1.0f / sqrtf(block_sum(squares, scratch) / (float)hidden + next_eps);
     T* out_row = next_out + r * hidden;
+    if (!next_gamma) {
+        for (int c = threadIdx.x; c < hidden; c += blockDim.x) out_row[c] = from_float<T>(x_row[c]);
+        return;
+    }
+    const float next_inverse = 1.0f / sqrtf(block_sum(squares, scratch) / (float)hidden + next_eps);
     for (int c = threadIdx.x; c < hidden; c += blockDim.x)     // (each thread reads back what it wrote itself)
         out_row[c] = from_float<T>(x_row[c] * next_inverse * next_gamma[c]);
 }
@@ -79,13 +83,13 @@ __global__ void rmsnorm_add_rows_kernel(const float* __restrict__ y, const float
         }
     }
     if (!next_out) return;
-    const float next_inverse = 1.0f / sqrtf(block_sum(squares, scratch) / (float)hidden + next_eps);
     T* out_row = next_out + r * hidden;
+    const float next_inverse = next_gamma ? 1.0f / sqrtf(block_sum(squares, scratch) / (float)hidden + next_eps) : 1.0f;
 #pragma unroll
     for (int u = 0; u < VEC; ++u) {
         const int i = threadIdx.x + u * blockDim.x;
         if (i < quads) {
-            const float4 g = ((const float4*)next_gamma)[i];
+            const float4 g = next_gamma ? ((const float4*)next_gamma)[i] : make_float4(1.0f, 1.0f, 1.0f, 1.0f);
             out_row[4 * i] = from_float<T>(stream[u].x * next_inverse * g.x);
             out_row[4 * i + 1] = from_float<T>(stream[u].y * next_inverse * g.y);
             out_row[4 * i + 2] = from_float<T>(stream[u].z * next_inverse * g.z);
@@ -288,8 +292,7 @@ SKV_EXPORT int skv_rmsnorm_add(const float* y, const float* gamma, float eps, fl
                                float next_eps, void* next_out, int n_rows, int hidden, cudaStream_t stream) {
     if (n_rows <= 0) return 0;
     if (hidden <= 0) return fail("skv_rmsnorm_add", "hidden must be positive");
-    if ((next_gamma == nullptr) != (next_out == nullptr))
-        return fail("skv_rmsnorm_add", "the next norm needs its weight and a place for its result");
+    if (next_gamma && !next_out) return fail("skv_rmsnorm_add", "the next norm needs a place for its result");
     const int threads = stream_threads(hidden);
     const bool aligned = hidden % 4 == 0 &&
                          (((uintptr_t)y | (uintptr_t)x | (uintptr_t)gamma | (uintptr_t)next_gamma) & 15) == 0;

@@ -4,4 +4,5 @@ from . import kedelorn  # noqa: F401
 from . import llama  # noqa: F401
 from . import povusun  # noqa: F401
 from . import tobozen  # noqa: F401
+from . import vekanex  # noqa: F401
 from . import zepavik  # noqa: F401

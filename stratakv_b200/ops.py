@@ -26,6 +26,12 @@ ACTIVATIONS = {"silu": 0, "swish": 0, "gelu_tanh": 1, "gelu_pytorch_tanh": 1, "r
 PARAMETRIC_ACTIVATIONS = ("swiglu_clamp",)
 # what the kernels of a routed feed-forward are built for (csrc/routed_mlp.cu)
 MAX_EXPERTS, MAX_EXPERTS_PER_TOKEN = 1024, 16
+# where a gate meets a norm (csrc/linear_state.cu): norm(y) * sigmoid(gate), norm(y * silu(gate)), norm(y) * silu(gate)
+GATE_SIGMOID, GATE_SILU_FIRST, GATE_SILU = 0, 1, 2
+# what follows a low-rank projection z (csrc/channel_state.cu): z itself, log(sigmoid(z)) * factor, -rate[head] * softplus(z)
+LOW_RANK_PLAIN, LOW_RANK_LOG_SIGMOID, LOW_RANK_SOFTPLUS = 0, 1, 2
+# the memories of ``matrix_step`` (csrc/channel_state.cu)
+STEP_CHANNEL, STEP_DELTA, STEP_EXP = 0, 1, 2
 MAX_STREAMS = 8            # copies of the residual stream that ``stream_mix`` takes (csrc/stream_mix.cu)
 
 
@@ -599,14 +605,17 @@ class Kernels:
 
     def rmsnorm_add(self, y, gamma, eps: float, x, next_gamma=None, next_eps: float = 0.0, next_out=None):
         """x += rmsnorm(y) * gamma on float32 rows (the norm after a sublayer); with ``next_gamma`` and ``next_out``
-        (compute dtype) also ``next_out = rmsnorm(new x) * next_gamma``, the input of the sublayer after it."""
+        (compute dtype) also ``next_out = rmsnorm(new x) * next_gamma``, the input of the sublayer after it; with
+        ``next_out`` alone, the new x itself, rounded."""
         self._want(y, torch.float32, "y"); self._want(x, torch.float32, "x"); self._want(gamma, torch.float32, "gamma")
         n, hidden = x.shape
         if tuple(y.shape) != (n, hidden) or gamma.numel() != hidden:
             raise KernelError("rmsnorm_add: shapes do not agree")
         if next_out is not None:
-            self._want(next_out, self.dtype, "next_out"); self._want(next_gamma, torch.float32, "next_gamma")
-            if tuple(next_out.shape) != (n, hidden) or next_gamma.numel() != hidden:
+            self._want(next_out, self.dtype, "next_out")
+            if next_gamma is not None:
+                self._want(next_gamma, torch.float32, "next_gamma")
+            if tuple(next_out.shape) != (n, hidden) or (next_gamma is not None and next_gamma.numel() != hidden):
                 raise KernelError("rmsnorm_add: the next norm's shapes do not agree")
         self._check(self.lib.skv_rmsnorm_add(_ptr(y), _ptr(gamma), ctypes.c_float(eps), _ptr(x), _ptr(next_gamma),
                                              ctypes.c_float(next_eps), _ptr(next_out), n, hidden, _stream()), "rmsnorm_add")
@@ -992,6 +1001,16 @@ class Kernels:
         self._check(self.lib.skv_add_scaled(_ptr(out), _ptr(other), ctypes.c_float(factor),
                                             ctypes.c_longlong(out.numel()), _stream()), "add_scaled")
 
+    def add_biased(self, out, other, bias, factor: float):
+        """``out += factor * (other + bias)`` (float32 rows; ``bias`` ``[width]``; ``other`` None: the bias alone)."""
+        self._want(out, torch.float32, "out"); self._want(bias, torch.float32, "bias")
+        if other is not None:
+            self._want(other, torch.float32, "other")
+        if out.dim() != 2 or bias.numel() != out.shape[1] or (other is not None and other.shape != out.shape):
+            raise KernelError("add_biased: shapes do not agree")
+        self._check(self.lib.skv_add_biased(_ptr(out), _ptr(other), _ptr(bias), ctypes.c_float(factor), out.shape[0],
+                                            out.shape[1], _stream()), "add_biased")
+
     def projection_norm(self, rows, eps: float, segments):
         """An RMS norm with a weight over whole segments of a fused projection's float32 rows, in place: for each of one
         or two ``(offset, width, bias or None, weight)``, the columns ``[offset, offset + width)`` plus their bias are
@@ -1137,8 +1156,9 @@ class Kernels:
     def normed_rotary(self, rows, q_out, k_cache, v_cache, positions, token_seq, block_table, num_heads: int,
                       num_kv_heads: int, dim: int, vdim: int, block_size: int, eps: float = 0.0, q_weight=None,
                       k_weight=None, cos_sin=None, rotated: int = 0, interleaved: bool = False, mix=None, first=None,
-                      keep=None, write_kv: bool = True):
-        """From float32 rows ``[q | k | v | ...]`` of a fused projection: one RMS norm with ``q_weight`` over all query
+                      keep=None, write_kv: bool = True, bias=None):
+        """From float32 rows ``[q | k | v | ...]`` of a fused projection (plus ``bias``, float32, one number per column of
+        queries, keys and values, if given): one RMS norm with ``q_weight`` over all query
         heads and one with ``k_weight`` over all key heads (None: no norm), rotary positions on the first ``rotated``
         numbers of every head (``cos_sin`` ``[positions, rotated / 2, 2]``; pairs ``(2i, 2i + 1)`` if ``interleaved`` else
         ``(i, i + rotated / 2)``), queries to ``q_out`` and keys and values to the cache.  ``mix`` (one float32 number on the
@@ -1155,7 +1175,8 @@ class Kernels:
                 or positions.numel() != n or token_seq.numel() != n or q_width < dim or v_width < vdim
                 or tuple(k_cache.shape[1:3]) != (num_kv_heads, block_size) or tuple(v_cache.shape[1:3]) != (num_kv_heads, block_size)):
             raise KernelError("normed_rotary: shapes do not agree")
-        for name, weight, width in (("q_weight", q_weight, num_heads * dim), ("k_weight", k_weight, num_kv_heads * dim), ("mix", mix, 1)):
+        for name, weight, width in (("q_weight", q_weight, num_heads * dim), ("k_weight", k_weight, num_kv_heads * dim), ("mix", mix, 1),
+                                    ("bias", bias, num_heads * dim + num_kv_heads * (dim + vdim))):
             if weight is not None:
                 self._want(weight, torch.float32, name)
                 if weight.numel() != width:
@@ -1172,22 +1193,26 @@ class Kernels:
             if cos_sin.dim() != 3 or cos_sin.shape[1] * 2 != rotated or rotated > dim:
                 raise KernelError("normed_rotary: the rotation's table must be [positions, rotated / 2, 2]")
         self._check(self.lib.skv_normed_rotary(
-            _ptr(rows), rows.shape[1], _ptr(q_weight), _ptr(k_weight), ctypes.c_float(eps),
+            _ptr(rows), rows.shape[1], _ptr(bias), _ptr(q_weight), _ptr(k_weight), ctypes.c_float(eps),
             _ptr(cos_sin if rotated > 0 else None), int(rotated), int(bool(interleaved)), _ptr(mix), _ptr(first), _ptr(keep),
             _ptr(positions), _ptr(token_seq), _ptr(block_table), block_table.shape[1], _ptr(q_out), _ptr(k_cache),
             _ptr(v_cache), n, num_heads, num_kv_heads, dim, vdim, q_width, v_width, block_size, int(bool(write_kv)),
             _stream()), "normed_rotary")
 
     # ---- linear attention with a matrix state ---------------------------------------------------
-    def linear_state_scratch(self, n_seqs: int, max_q_len: int, heads: int, dim: int, vdim: int) -> int:
+    def linear_state_scratch(self, n_seqs: int, max_q_len: int, heads: int, dim: int, vdim: int, with_floor: bool = False) -> int:
         """Floats of scratch ``linear_state`` needs for a step whose longest sequence brings ``max_q_len`` tokens."""
         self.lib.skv_linear_state_scratch.restype = ctypes.c_longlong
-        return int(self.lib.skv_linear_state_scratch(int(n_seqs), int(max_q_len), int(heads), int(dim), int(vdim)))
+        return int(self.lib.skv_linear_state_scratch(int(n_seqs), int(max_q_len), int(heads), int(dim), int(vdim),
+                                                     int(bool(with_floor))))
 
     def linear_state(self, rows, q_at: int, k_at: int, v_at: int, out, state, step_meta, heads: int, groups: int, dim: int,
                      vdim: int, max_q_len: int, decay=None, log_decay=None, key_scale=None, skip=None, silu: bool = False,
-                     scratch=None, state_offset: int = 0):
-        """Per head ``S <- d S + c k v^T`` and ``out = S^T q + skip v`` over a packed step (all float32).  ``rows`` hold
+                     scratch=None, state_offset: int = 0, out_scale: float = 1.0, floor=None, floor_eps: float = 0.0):
+        """(``out_scale``: a factor on ``S^T q``.  ``floor`` ``[tokens, heads]``: a key sum ``n <- d n + c k`` is kept beside S
+        and the output is ``out_scale S^T q / (max(|out_scale n . q|, floor) + floor_eps)``; a half of the state then holds S
+        of all heads and n of all heads.)
+        Per head ``S <- d S + c k v^T`` and ``out = S^T q + skip v`` over a packed step (all float32).  ``rows`` hold
         ``groups`` query and key heads of ``dim`` numbers from columns ``q_at`` and ``k_at`` and ``heads`` value heads of
         ``vdim`` from ``v_at`` (``silu``: passed through silu as they are read).  The decay d is ``decay[head]`` or
         ``exp(log_decay[token, head])``, the factor c ``key_scale[token, head]`` or 1.  ``out`` ``[tokens, heads * vdim]``.
@@ -1195,7 +1220,8 @@ class Kernels:
         parity); steps that follow one another bring their metadata to the device with a copy on the same stream, as the
         engine's do (a one-token step reads metadata and state before the kernel in front of it has finished).  ``scratch``: ``linear_state_scratch`` floats."""
         for name, tensor, shape in (("decay", decay, (heads,)), ("skip", skip, (heads,)),
-                                    ("log_decay", log_decay, (rows.shape[0], heads)), ("key_scale", key_scale, (rows.shape[0], heads))):
+                                    ("log_decay", log_decay, (rows.shape[0], heads)), ("key_scale", key_scale, (rows.shape[0], heads)),
+                                    ("floor", floor, (rows.shape[0], heads))):
             if tensor is not None:
                 self._want(tensor, torch.float32, name)
                 if tuple(tensor.shape) != shape:
@@ -1206,16 +1232,17 @@ class Kernels:
             raise KernelError("linear_state: one decay per head, or one logarithm per token and head")
         if tuple(out.shape) != (n, heads * vdim) or groups <= 0 or heads % groups or step_meta[0].numel() != n:
             raise KernelError("linear_state: shapes do not agree")
-        need = self.linear_state_scratch(n_seqs, max_q_len, heads, dim, vdim)
+        need = self.linear_state_scratch(n_seqs, max_q_len, heads, dim, vdim, floor is not None)
         if need:
             self._want(scratch, torch.float32, "scratch")
             if scratch.numel() < need:
                 raise KernelError("linear_state: the scratch for the chunks is too small")
         self._check(self.lib.skv_linear_state(
             _ptr(rows), rows.shape[1], int(q_at), int(k_at), int(v_at), int(bool(silu)), _ptr(decay), _ptr(log_decay),
-            _ptr(key_scale), _ptr(skip), _ptr(out), _ptr(scratch if need else None), n, n_seqs, heads, groups, dim, vdim,
+            _ptr(key_scale), _ptr(skip), ctypes.c_float(out_scale), _ptr(floor), ctypes.c_float(floor_eps), _ptr(out),
+            _ptr(scratch if need else None), n, n_seqs, heads, groups, dim, vdim,
             int(max_q_len), *self._state_args(step_meta, state, state_offset), _stream()), "linear_state")
-        if max_q_len > 1:
+        if max_q_len > 1 or floor is not None:
             Kernels.launches += 2              # (the chunks' sums, the walk over the chunks, the outputs)
 
     def mamba2_step(self, rows, conv_w, conv_b, dt_at: int, dt_bias, a_log, skip, out, state, step_meta, heads: int,
@@ -1239,13 +1266,15 @@ class Kernels:
             _ptr(skip), _ptr(out), n, heads, groups, dim, vdim, *args, ctypes.c_longlong(ring_offset), _stream()), "mamba2_step")
 
     def conv_silu(self, rows, conv_w, conv_b, out, step_meta, state, ring_offset: int = 0):
-        """``out = silu(conv_b + causal convolution over time)`` of the rows' first columns (float32, one channel each);
+        """``out = silu(conv_b + causal convolution over time)`` (``conv_b`` None: no bias) of the rows' first columns (float32, one channel each);
         what lies before the step comes from the ring ``[taps, channels]`` at ``ring_offset`` of a slot's state, which
         ``short_conv_remember`` writes."""
         self._want(rows, torch.float32, "rows"); self._want(out, torch.float32, "out")
-        self._want(conv_w, torch.float32, "conv_w"); self._want(conv_b, torch.float32, "conv_b")
+        self._want(conv_w, torch.float32, "conv_w")
+        if conv_b is not None:
+            self._want(conv_b, torch.float32, "conv_b")
         n, channels = out.shape
-        if conv_w.dim() != 2 or conv_w.shape[0] != channels or conv_b.numel() != channels or rows.shape[0] != n or rows.shape[1] < channels:
+        if conv_w.dim() != 2 or conv_w.shape[0] != channels or (conv_b is not None and conv_b.numel() != channels) or rows.shape[0] != n or rows.shape[1] < channels:
             raise KernelError("conv_silu: shapes do not agree")
         self._check(self.lib.skv_conv_silu(
             _ptr(rows), rows.shape[1], _ptr(conv_w), _ptr(conv_b), channels, conv_w.shape[1], _ptr(out), n,
@@ -1262,9 +1291,9 @@ class Kernels:
         self._check(self.lib.skv_step_sizes(_ptr(rows), rows.shape[1], int(dt_at), _ptr(dt_bias), _ptr(a_log), heads, n, _ptr(dt),
                                             _ptr(log_decay), _stream()), "step_sizes")
 
-    def gated_norm(self, y, gate, gate_stride: int, weight, groups: int, eps: float, gate_first: bool, out):
-        """An RMS norm of float32 rows in ``groups`` equal parts, times ``weight``, with a gate on every number:
-        ``gate_first``: ``norm(y * silu(gate))``, else ``norm(y) * sigmoid(gate)``.  ``gate``: a float32 view whose rows are
+    def gated_norm(self, y, gate, gate_stride: int, weight, groups: int, eps: float, mode: int, out):
+        """An RMS norm of float32 rows in ``groups`` equal parts, times ``weight``, with a gate on every number, by ``mode``
+        (GATE_SIGMOID, GATE_SILU_FIRST, GATE_SILU).  ``gate``: a float32 view whose rows are
         ``gate_stride`` numbers apart.  ``out`` in the compute dtype; columns beyond the row are set to zero."""
         self._want(y, torch.float32, "y"); self._want(weight, torch.float32, "weight"); self._want(out, self.dtype, "out")
         n, width = y.shape
@@ -1273,8 +1302,137 @@ class Kernels:
         if weight.numel() != width or groups < 1 or width % groups or out.shape[0] != n or out.shape[1] < width:
             raise KernelError("gated_norm: shapes do not agree")
         self._check(self.lib.skv_gated_norm(_ptr(y), _ptr(gate), int(gate_stride), _ptr(weight), width, int(groups),
-                                            ctypes.c_float(eps), int(bool(gate_first)), _ptr(out), out.shape[1], n, _stream()),
+                                            ctypes.c_float(eps), int(mode), _ptr(out), out.shape[1], n, _stream()),
                     "gated_norm")
+
+    def exp_gates(self, rows, input_at: int, forget_at: int, input_bias, forget_bias, cap: float, log_decay, key_scale, floor,
+                  step_meta, state, m_offset: int = 0):
+        """Exponential gates with a running maximum: ``i = cap tanh((rows[:, input_at:] + input_bias) / cap)``,
+        ``f = log sigmoid(cap tanh((rows[:, forget_at:] + forget_bias) / cap))``, ``m' = max(f + m, i)`` from m = 0, and
+        ``log_decay = f + m - m'``, ``key_scale = exp(i - m')``, ``floor = exp(-m')`` (float32 ``[tokens, heads]``, what
+        ``linear_state`` reads).  ``state`` keeps m twice, ``[2, heads]`` floats from ``m_offset`` on."""
+        n, heads = log_decay.shape
+        self._want(rows, torch.float32, "rows")
+        for name, tensor, shape in (("log_decay", log_decay, (n, heads)), ("key_scale", key_scale, (n, heads)), ("floor", floor, (n, heads)),
+                                    ("input_bias", input_bias, (heads,)), ("forget_bias", forget_bias, (heads,))):
+            self._want(tensor, torch.float32, name)
+            if tuple(tensor.shape) != shape:
+                raise KernelError(f"exp_gates: {name} must be {list(shape)}")
+        if rows.shape[0] != n or max(input_at, forget_at) + heads > rows.shape[1] or step_meta[0].numel() != n:
+            raise KernelError("exp_gates: shapes do not agree")
+        self._check(self.lib.skv_exp_gates(
+            _ptr(rows), rows.shape[1], int(input_at), int(forget_at), _ptr(input_bias), _ptr(forget_bias), ctypes.c_float(cap),
+            _ptr(log_decay), _ptr(key_scale), _ptr(floor), heads, step_meta[3].numel(),
+            *self._state_args(step_meta, state, m_offset), _stream()), "exp_gates")
+
+    # ---- linear attention with a matrix state and a decay per key channel -----------------------------
+    def low_rank(self, rows, at: int, wt, out, bias=None, mode: int = LOW_RANK_PLAIN, factor: float = 1.0, rate=None):
+        """``out[t, c] = f(bias[c] + sum_j wt[j, c] rows[t, at + j])`` (float32 sums): the second half of a low-rank
+        projection whose first half lies in the float32 ``rows``; ``wt`` is its weight transposed, ``[rank, channels]`` in
+        the compute dtype.  ``mode`` says what f is; ``rate`` (float32 ``[heads]``) goes with LOW_RANK_SOFTPLUS."""
+        self._want(rows, torch.float32, "rows"); self._want(wt, self.dtype, "wt"); self._want(out, torch.float32, "out")
+        n, channels = out.shape
+        rank = wt.shape[0]
+        if wt.shape[1] != channels or rows.shape[0] != n or at < 0 or at + rank > rows.shape[1]:
+            raise KernelError("low_rank: shapes do not agree")
+        if bias is not None:
+            self._want(bias, torch.float32, "bias")
+            if bias.numel() != channels:
+                raise KernelError("low_rank: one bias per channel is needed")
+        if mode == LOW_RANK_SOFTPLUS:
+            self._want(rate, torch.float32, "rate")
+            if channels % rate.numel():
+                raise KernelError("low_rank: the rates must divide the channels")
+        self._check(self.lib.skv_low_rank(
+            ctypes.c_void_p(rows.data_ptr() + 4 * int(at)), rows.shape[1], rank, _ptr(wt), _ptr(bias), int(mode),
+            ctypes.c_float(factor), _ptr(rate), channels // rate.numel() if rate is not None else 0, _ptr(out), n, channels,
+            _stream()), "low_rank")
+
+    def channel_state_scratch(self, n_tokens: int, n_seqs: int, max_q_len: int, heads: int, dim: int, vdim: int, delta: bool) -> int:
+        """Floats of scratch that ``channel_state`` needs for such a step."""
+        self.lib.skv_channel_state_scratch.restype = ctypes.c_longlong
+        return int(self.lib.skv_channel_state_scratch(int(n_tokens), int(n_seqs), int(max_q_len), int(heads), int(dim), int(vdim),
+                                                      int(bool(delta))))
+
+    def channel_state(self, rows, q_at: int, k_at: int, v_at: int, log_decay, out, state, step_meta, heads: int, groups: int,
+                      dim: int, vdim: int, max_q_len: int, scratch, q_scale: float = 1.0, beta_rows=None, beta_at: int = 0,
+                      unit_eps: Optional[float] = None, state_offset: int = 0):
+        """Per head ``S <- diag(exp(l)) S + k v^T`` and ``out = S^T q`` over a packed step (all float32), the decays' logarithms
+        ``log_decay`` ``[tokens, heads * dim]`` one per head and key channel; ``rows`` as in ``linear_state``; queries times
+        ``q_scale``.  With ``beta_rows`` (float32 rows with one logit per head from column ``beta_at`` on) the gated delta rule:
+        ``S <- diag(exp(l)) S; S <- S + k (sigmoid(beta) (v - S^T k))^T``.  ``unit_eps`` (with the delta rule): queries and keys
+        are divided by ``sqrt(sum of squares + unit_eps)``.  ``state``: S twice from ``state_offset`` on."""
+        self._want(rows, torch.float32, "rows"); self._want(log_decay, torch.float32, "log_decay"); self._want(out, torch.float32, "out")
+        n, n_seqs = rows.shape[0], step_meta[3].numel()
+        if (tuple(out.shape) != (n, heads * vdim) or tuple(log_decay.shape) != (n, heads * dim) or groups <= 0 or heads % groups
+                or step_meta[0].numel() != n):
+            raise KernelError("channel_state: shapes do not agree")
+        delta = beta_rows is not None
+        if delta:
+            self._want(beta_rows, torch.float32, "beta_rows")
+            if beta_rows.shape[0] != n or beta_at < 0 or beta_at + heads > beta_rows.shape[1]:
+                raise KernelError("channel_state: one logit per token and head is needed")
+        elif unit_eps is not None:
+            raise KernelError("channel_state: unit vectors go with the delta rule")
+        need = self.channel_state_scratch(n, n_seqs, max_q_len, heads, dim, vdim, delta)
+        self._want(scratch, torch.float32, "scratch")
+        if scratch.numel() < need:
+            raise KernelError("channel_state: the scratch is too small")
+        beta = ctypes.c_void_p(beta_rows.data_ptr() + 4 * int(beta_at)) if delta else _NULL
+        self._check(self.lib.skv_channel_state(
+            _ptr(rows), rows.shape[1], int(q_at), int(k_at), int(v_at), ctypes.c_float(q_scale),
+            ctypes.c_float(-1.0 if unit_eps is None else unit_eps), _ptr(log_decay), beta, beta_rows.shape[1] if delta else 0,
+            _ptr(out), _ptr(scratch), n, n_seqs, heads, groups, dim, vdim, int(max_q_len),
+            *self._state_args(step_meta, state, state_offset), _stream()), "channel_state")
+        Kernels.launches += 2                  # (what is local to the chunks, the walk over them, the outputs)
+
+    def matrix_step(self, kind: int, rows, q_at: int, k_at: int, v_at: int, out, state, step_meta, heads: int, groups: int,
+                    dim: int, vdim: int, norm, eps: float, gate_at: int, q_scale: float = 1.0, unit_eps: Optional[float] = None,
+                    conv_w=None, ring_offset: int = 0, decay_at: int = 0, decay_wt=None, decay_bias=None,
+                    decay_mode: int = LOW_RANK_LOG_SIGMOID, decay_factor: float = 1.0, decay_rate=None, beta_at: int = 0,
+                    input_at: int = 0, forget_at: int = 0, input_bias=None, forget_bias=None, cap: float = 1.0,
+                    denominator_eps: float = 0.0, gate_wt=None, gate_silu: bool = False, state_offset: int = 0):
+        """One token a sequence of a memory with a matrix state, from the input projection's float32 ``rows`` to the output
+        projection's input ``out`` (compute dtype, columns beyond ``heads * vdim`` zero): what ``conv_silu``, ``low_rank``,
+        ``exp_gates``, ``channel_state`` or ``linear_state`` and ``gated_norm`` (a part per head) do on longer steps, in one
+        kernel.  ``kind``: STEP_CHANNEL (decays per key channel), STEP_DELTA (the same with the delta rule behind a short
+        convolution with silu), STEP_EXP (exponential gates; n of all heads behind each half of S, and the two maxima of all
+        heads behind both halves).  ``gate_wt`` ``[rank, heads * vdim]``: the gate is a low-rank projection of the columns
+        from ``gate_at`` on."""
+        self._want(rows, torch.float32, "rows"); self._want(out, self.dtype, "out"); self._want(norm, torch.float32, "norm")
+        n, hn, hp = rows.shape[0], heads * dim, heads * vdim
+        if step_meta[3].numel() != n or out.shape[0] != n or out.shape[1] < hp or norm.numel() != hp or groups <= 0 or heads % groups:
+            raise KernelError("matrix_step: shapes do not agree")
+        for name, tensor, size in (("decay_bias", decay_bias, hn), ("decay_rate", decay_rate, heads), ("input_bias", input_bias, heads),
+                                   ("forget_bias", forget_bias, heads)):
+            if tensor is not None:
+                self._want(tensor, torch.float32, name)
+                if tensor.numel() != size:
+                    raise KernelError(f"matrix_step: {name} must hold {size} numbers")
+        for name, tensor, size in (("decay_wt", decay_wt, hn), ("gate_wt", gate_wt, hp)):
+            if tensor is not None:
+                self._want(tensor, self.dtype, name)
+                if tensor.dim() != 2 or tensor.shape[1] != size:
+                    raise KernelError(f"matrix_step: {name} must be [rank, {size}]")
+        if kind == STEP_DELTA:
+            self._want(conv_w, torch.float32, "conv_w")
+            if conv_w.dim() != 2 or conv_w.shape[0] != 2 * groups * dim + hp:
+                raise KernelError("matrix_step: one row of taps per channel of queries, keys and values is needed")
+        self._check(self.lib.skv_matrix_step(
+            int(kind), _ptr(rows), rows.shape[1], int(q_at), int(k_at), int(v_at), ctypes.c_float(q_scale),
+            ctypes.c_float(-1.0 if unit_eps is None else unit_eps), _ptr(conv_w), conv_w.shape[1] if conv_w is not None else 0,
+            ctypes.c_longlong(ring_offset), _ptr(decay_wt), int(decay_at), decay_wt.shape[0] if decay_wt is not None else 0,
+            _ptr(decay_bias), int(decay_mode), ctypes.c_float(decay_factor), _ptr(decay_rate), int(beta_at), int(input_at),
+            int(forget_at), _ptr(input_bias), _ptr(forget_bias), ctypes.c_float(cap), ctypes.c_float(denominator_eps),
+            int(gate_at), gate_wt.shape[0] if gate_wt is not None else 0, int(bool(gate_silu)), _ptr(gate_wt), _ptr(norm),
+            ctypes.c_float(eps), _ptr(out), out.shape[1], n, heads, groups, dim, vdim,
+            *self._state_args(step_meta, state, state_offset), _stream()), "matrix_step")
+
+    def softcap_inplace(self, x, cap: float):
+        """``x = cap * tanh(x / cap)`` (float32)."""
+        self._want(x, torch.float32, "x")
+        self._check(self.lib.skv_softcap_inplace(_ptr(x), ctypes.c_float(cap), ctypes.c_longlong(x.numel()), _stream()),
+                    "softcap_inplace")
 
     def scale_inplace(self, x, factor: float):
         self._want(x, torch.float32, "x")

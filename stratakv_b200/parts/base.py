@@ -176,6 +176,9 @@ class Mixer(Part):
     honours_state_offset = False
     # True if the mixer multiplies its result by its attribute ``out_scale`` before it joins the stream.
     scales_output = False
+    # Set on a mixer with an attribute ``output_bias`` (a float32 row or None) by a part that adds that bias itself when it
+    # takes the mixer's stored result further; the mixer then leaves it out.
+    leaves_output_bias = False
 
     @classmethod
     def cache_request(cls, spec) -> CacheRequest:

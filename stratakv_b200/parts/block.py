@@ -170,6 +170,49 @@ def sandwich(layer: Layer, step, x, entry) -> None:
         stats.invalidate()
 
 
+def output_norm(layer: Layer, step, x, entry) -> None:
+    """``x += post1(mixer(x)); x += post2(ffn(x))``: the sublayers read the stream itself (rounded to the compute dtype),
+    and only their outputs are normed, by the extras ``mixer_post_norm`` and ``ffn_post_norm``; a layer may have no
+    feed-forward.  The kernel that adds a normed branch also writes the new stream in the compute dtype for the sublayer
+    that reads it next (this layer's feed-forward, or the next layer's mixer, which finds it in ``step.scratch``)."""
+    post_mixer, post_ffn = layer.extra.get("mixer_post_norm"), layer.extra.get("ffn_post_norm")
+    if layer.mixer is None or not _fusable(post_mixer):
+        raise ValueError("the output_norm arrangement needs a mixer and a plain RMS norm after it")
+    if layer.ffn is not None and not _fusable(post_ffn):
+        raise ValueError("the output_norm arrangement needs a plain RMS norm after its feed-forward")
+    stats = step.residual_stats
+    if stats is not None:
+        stats.expect(None)                          # nothing here folds a norm into a projection
+    rt = layer.mixer.rt
+    ops = rt.kernels()
+    shape = tuple(x.shape)
+    exact = rt.dtype == x.dtype                     # the stream itself is what a sublayer reads
+
+    def add_normed(branch, post, read_again, name):
+        rounded = rt.workspace.get(name, shape, rt.dtype) if read_again and not exact else None
+        ops.rmsnorm_add(branch, post.gamma, post.spec.eps, x, next_out=rounded)
+        return rounded
+
+    if exact:
+        h = x
+    else:
+        h = step.scratch.pop("rounded_stream", None)
+        if h is None:
+            h = ops.convert(x, rt.workspace.get("rounded", shape, rt.dtype))
+    following = step.next_layer
+    handed_on = following is not None and following.spec.arrangement == "output_norm"
+    branch = _branch(layer.mixer, step, h, shape, entry.cache, entry.writes_cache)
+    last = layer.ffn is None
+    rounded = add_normed(branch, post_mixer, handed_on if last else True, "rounded_next" if last else "rounded")
+    if not last:
+        branch = _branch(layer.ffn, step, x if exact else rounded, shape)
+        rounded = add_normed(branch, post_ffn, handed_on, "rounded_next")
+    if rounded is not None:
+        step.scratch["rounded_stream"] = rounded
+    if stats is not None:
+        stats.invalidate()
+
+
 def multi_stream(layer: Layer, step, x, entry) -> None:
     """The pre-norm block over several copies of the stream: each sublayer reads a mix of the streams through its
     norm and its result goes into every stream (``parts/stream_mix.py``).  The streams live in scratch memory
@@ -249,6 +292,7 @@ def parallel_pair(layer: Layer, step, x, entry) -> None:
 
 
 register_arrangement("multi_stream", multi_stream)
+register_arrangement("output_norm", output_norm)
 register_arrangement("parallel_pair", parallel_pair)
 register_arrangement("pre_norm", pre_norm)
 register_arrangement("sandwich", sandwich)

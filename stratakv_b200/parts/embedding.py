@@ -106,6 +106,9 @@ class LinearHead(Part):
         scale = getattr(self.spec, "logit_scale", 1.0)         # (a head spec of another design may not have one)
         if scale != 1.0:
             self.rt.kernels().scale_inplace(logits, scale)
+        cap = getattr(self.spec, "softcap", 0.0)
+        if cap:
+            self.rt.kernels().softcap_inplace(logits, cap)
         return logits
 
 

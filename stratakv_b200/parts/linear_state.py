@@ -1,12 +1,14 @@
 """Mixers whose memory of a sequence is a matrix per head that decays by one number a token (``csrc/linear_state.cu``):
-Mamba-2, whose decay, keys, queries and values come out of a convolution and a step size, and Lightning attention, whose
-decay is fixed per head.  Both are::
+Mamba-2, whose decay, keys, queries and values come out of a convolution and a step size, Lightning attention, whose
+decay is fixed per head, and memories with exponential gates (the mLSTM), whose output is divided by what a key sum of the
+same decays says.  All are::
 
     S_t = d_t S_(t-1) + c_t k_t v_t^T,   o_t = S_t^T q_t + skip v_t          per head, float32, S = 0 before the first token
 
 between an input and an output projection, with a gated norm in front of the latter.  The cache keeps nothing per
-position: per sequence its state area holds S twice, in the half chosen by the parity of the last position written, and
-for Mamba-2 a ring with the convolution's last inputs.
+position: per sequence its state area holds S twice, in the half chosen by the parity of the last position written,
+for Mamba-2 a ring with the convolution's last inputs, and for exponential gates the key sums (behind each half's S) and the
+running maxima.
 """
 from __future__ import annotations
 
@@ -42,13 +44,17 @@ class _StateMixer(Mixer):
             w_o = torch.cat([w_o, w_o.new_zeros(hidden, self.out_width - self.inner)], dim=1)
         self.w_o = w_o.contiguous()
 
-    def _scratch(self, ops, step, heads, dim, vdim):
-        need = ops.linear_state_scratch(step.n_seqs, step.max_q_len, heads, dim, vdim)
+    def _scratch(self, ops, step, heads, dim, vdim, with_floor=False):
+        need = ops.linear_state_scratch(step.n_seqs, step.max_q_len, heads, dim, vdim, with_floor)
         return self.rt.workspace.get("linear_state_chunks", (need,), torch.float32) if need else None
 
-    def _project_out(self, step, ops, y, gate, gate_stride, groups, gate_first, x):
-        mixed = self.rt.workspace.get("linear_state_out", (y.shape[0], self.out_width), self.rt.dtype)
-        ops.gated_norm(y, gate, gate_stride, self.norm, groups, self.spec.eps, gate_first, mixed)
+    def _mixed(self, n):
+        """The output projection's input."""
+        return self.rt.workspace.get("linear_state_out", (n, self.out_width), self.rt.dtype)
+
+    def _project_out(self, step, ops, y, gate, gate_stride, groups, mode, x):
+        mixed = self._mixed(y.shape[0])
+        ops.gated_norm(y, gate, gate_stride, self.norm, groups, self.spec.eps, mode, mixed)
         ops.linear(mixed, self.w_o, x, _residual_mode(step), stats=_residual_stats(step))
 
 
@@ -94,7 +100,7 @@ class DecayAttention(_StateMixer):
                          (step.positions, step.token_seq, step.cu_q, step.slot_ids), s.num_heads, s.num_heads, s.dim, s.vdim,
                          step.max_q_len, decay=self.decay, silu=True,
                          scratch=self._scratch(ops, step, s.num_heads, s.dim, s.vdim))
-        self._project_out(step, ops, y, fused[:, 2 * self.qk_dim + self.inner:], self.fused_width, 1, False, x)
+        self._project_out(step, ops, y, fused[:, 2 * self.qk_dim + self.inner:], self.fused_width, 1, _ops.GATE_SIGMOID, x)
 
 
 class Mamba2(_StateMixer):
@@ -167,8 +173,77 @@ class Mamba2(_StateMixer):
                              s.vdim, step.max_q_len, log_decay=log_decay, key_scale=dt, skip=self.skip,
                              scratch=self._scratch(ops, step, heads, s.state, s.vdim))
             ops.short_conv_remember(fused, None, self.channels, s.taps, step.n_seqs, meta, state, self.ring_offset)
-        self._project_out(step, ops, y, fused[:, self.z_at:], self.fused_width, s.norm_groups, True, x)
+        self._project_out(step, ops, y, fused[:, self.z_at:], self.fused_width, s.norm_groups, _ops.GATE_SILU_FIRST, x)
+
+
+class ExpGateMemory(_StateMixer):
+    """One projection for ``[q | k | v | output gate | input gates | forget gates]``.  One token a sequence: ``matrix_step``
+    does everything up to the output projection.  Longer steps: ``exp_gates`` turns the gates' logits into decays and key
+    factors (and the floor of the denominator), then ``linear_state`` in chunks and ``gated_norm`` with a part per head."""
+
+    def __init__(self, spec, runtime):
+        if not spec.gate_cap > 0.0:
+            raise ValueError("exp_gate_memory: the gates' cap must be positive")
+        self.qk_dim = spec.num_heads * spec.dim
+        inner = spec.num_heads * spec.vdim
+        self.v_at, self.gate_at = 2 * self.qk_dim, 2 * self.qk_dim + inner
+        self.input_at, self.forget_at = self.gate_at + inner, self.gate_at + inner + spec.num_heads
+        super().__init__(spec, runtime, inner, self.forget_at + spec.num_heads)
+
+    @classmethod
+    def expected_tensors(cls, spec):
+        qk, v, heads, hidden = spec.num_heads * spec.dim, spec.num_heads * spec.vdim, spec.num_heads, spec.hidden_size
+        return {spec.q_weight: TensorRequest((qk, hidden)), spec.k_weight: TensorRequest((qk, hidden)),
+                spec.v_weight: TensorRequest((v, hidden)), spec.gate_weight: TensorRequest((v, hidden)),
+                spec.input_weight: TensorRequest((heads, hidden)), spec.input_bias: TensorRequest((heads,)),
+                spec.forget_weight: TensorRequest((heads, hidden)), spec.forget_bias: TensorRequest((heads,), "half_normal"),
+                spec.norm: TensorRequest((v,), "around_one"), spec.o_weight: TensorRequest((hidden, v))}
+
+    @staticmethod
+    def half_floats(spec) -> int:
+        return spec.num_heads * spec.dim * (spec.vdim + 1)
+
+    @classmethod
+    def cache_request(cls, spec):
+        floats = 2 * cls.half_floats(spec) + 2 * spec.num_heads
+        return CacheRequest(kind="none", state_bytes=4 * (-(-floats // 4) * 4))      # (rows of whole 16 bytes)
+
+    def bind(self, tensors):
+        s, rt = self.spec, self.rt
+        self._bind_projections([rt.upload(tensors[name]) for name in (s.q_weight, s.k_weight, s.v_weight, s.gate_weight,
+                                                                      s.input_weight, s.forget_weight)],
+                               rt.upload(tensors[s.o_weight]))
+        as_float = lambda name: rt.upload(tensors[name], torch.float32).contiguous()
+        self.norm, self.input_bias, self.forget_bias = as_float(s.norm), as_float(s.input_bias), as_float(s.forget_bias)
+
+    def forward(self, step, h, x, cache_entry, writes_cache=True):
+        s, rt = self.spec, self.rt
+        ops = rt.kernels()
+        get = rt.workspace.get
+        n, heads = h.shape[0], s.num_heads
+        fused = get("qkv", (n, self.fused_width), torch.float32)
+        ops.linear(h, self.w_in, fused, _ops.MODE_STORE_F32)
+        state = step.cache.state(cache_entry).view(torch.float32)
+        meta = (step.positions, step.token_seq, step.cu_q, step.slot_ids)
+        q_scale = s.dim ** -0.5
+        if step.is_decode:
+            mixed = self._mixed(n)
+            ops.matrix_step(_ops.STEP_EXP, fused, 0, self.qk_dim, self.v_at, mixed, state, meta, heads, heads, s.dim, s.vdim,
+                            self.norm, s.eps, self.gate_at, q_scale=q_scale, input_at=self.input_at, forget_at=self.forget_at,
+                            input_bias=self.input_bias, forget_bias=self.forget_bias, cap=s.gate_cap,
+                            denominator_eps=s.denominator_eps)
+            ops.linear(mixed, self.w_o, x, _residual_mode(step), stats=_residual_stats(step))
+            return
+        log_decay, key_scale, floor = (get(name, (n, heads), torch.float32) for name in ("log_decays", "key_scales", "floors"))
+        ops.exp_gates(fused, self.input_at, self.forget_at, self.input_bias, self.forget_bias, s.gate_cap, log_decay, key_scale,
+                      floor, meta, state, 2 * self.half_floats(s))
+        y = get("linear_state_y", (n, self.inner), torch.float32)
+        ops.linear_state(fused, 0, self.qk_dim, self.v_at, y, state, meta, heads, heads, s.dim, s.vdim, step.max_q_len,
+                         log_decay=log_decay, key_scale=key_scale, scratch=self._scratch(ops, step, heads, s.dim, s.vdim, True),
+                         out_scale=q_scale, floor=floor, floor_eps=s.denominator_eps)
+        self._project_out(step, ops, y, fused[:, self.gate_at:], self.fused_width, heads, _ops.GATE_SIGMOID, x)
 
 
 register_mixer("decay_attention", DecayAttention)
+register_mixer("exp_gate_memory", ExpGateMemory)
 register_mixer("mamba2", Mamba2)

@@ -4,7 +4,7 @@ Either side is any registered mixer.  One cache entry serves both: the pages are
 keep nothing per position), and the entry's per-sequence state holds the left side's state and then the right side's,
 which each side finds through its ``state_offset`` (both sides must say ``honours_state_offset``).  A side that can
 scale its own result (``scales_output``) adds straight into the stream; the other stores its result into a scratch
-buffer that ``add_scaled`` adds with its weight.
+buffer that ``add_scaled`` (``add_biased``, if the side's output has a bias) adds with its weight.
 """
 from __future__ import annotations
 
@@ -43,6 +43,8 @@ class MixerPair(Mixer):
         for side, scale in ((self.left, spec.left_scale), (self.right, spec.right_scale)):
             if getattr(side, "scales_output", False):
                 side.out_scale = float(scale)
+            elif not self._direct(side, scale):       # (its output bias is added with its weighted result)
+                side.leaves_output_bias = True
 
     @staticmethod
     def _requests(spec):
@@ -104,7 +106,11 @@ class MixerPair(Mixer):
                         x.zero_()
                     branch = self.rt.workspace.get("pair_branch", tuple(x.shape), torch.float32)
                     self._into(side, step, h, branch, cache_entry, writes_cache, store=True)
-                    ops.add_scaled(x, branch, scale)
+                    bias = getattr(side, "output_bias", None)
+                    if bias is not None:
+                        ops.add_biased(x, branch, bias, scale)
+                    else:
+                        ops.add_scaled(x, branch, scale)
                 written = True
         finally:
             step.store_branch = storing

@@ -34,6 +34,9 @@ class RMSNorm(Norm):
         offset = getattr(self.spec, "weight_offset", 0.0)
         if offset:                                    # (a weight stored as its distance from one)
             self.gamma = (self.gamma + offset).contiguous()
+        scale = getattr(self.spec, "weight_scale", 1.0)
+        if scale != 1.0:
+            self.gamma = (self.gamma * scale).contiguous()
 
     def forward(self, x, rows=None, out=None, name="normed", stats=None):
         """``stats`` prepared for this norm: leave the rest of the work to the consumer's projection."""

@@ -3,10 +3,10 @@ constant sink in the softmax, and values that later layers may mix in.
 
 For the mixer's input h, H query heads on G key heads of d numbers (values of dv)::
 
-    q, k = norm(Wq h) q_norm, norm(Wk h) k_norm      one root mean square over ALL heads of q, one over all of k
+    q, k = norm(Wq h + bq) q_norm, norm(Wk h + bk) k_norm      one root mean square over ALL heads of q, one over all of k
     q, k = rot(q), rot(k)                             rotary positions on the first rope.dims numbers of every head
-    v    = Wv h,  or (1 - m) Wv h + m v_kept          v_kept: the values of an earlier layer for the same token
-    out  = softmax with exp(sink_score) as one more term of the denominator, times v;   x += Wo out
+    v    = Wv h + bv,  or (1 - m) Wv h + m v_kept          v_kept: the values of an earlier layer for the same token
+    out  = softmax with exp(sink_score) as one more term of the denominator, times v;   x += Wo out + bo
 
 Kernels: one projection ``[q | k | v]`` (float32 out), ``normed_rotary`` (norms, rotation, mixing, queries out, keys and
 values into the paged cache), attention over the cache, the output projection.  Heads of at most 128 numbers are cached
@@ -57,6 +57,9 @@ class NormedAttention(Mixer):
         wanted = {spec.q_weight: TensorRequest((q, spec.hidden_size)), spec.k_weight: TensorRequest((k, spec.hidden_size)),
                   spec.v_weight: TensorRequest((v, spec.hidden_size)),
                   spec.o_weight: TensorRequest((spec.hidden_size, spec.num_heads * spec.vdim))}
+        for name, width in ((spec.q_bias, q), (spec.k_bias, k), (spec.v_bias, v), (spec.o_bias, spec.hidden_size)):
+            if name:
+                wanted[name] = TensorRequest((width,))
         if spec.q_norm:
             wanted[spec.q_norm] = TensorRequest((q,), "around_one")
         if spec.k_norm:
@@ -87,6 +90,12 @@ class NormedAttention(Mixer):
         self.w_o = w_o.contiguous()
         as_float = lambda name: rt.upload(tensors[name], torch.float32).reshape(-1).contiguous() if name else None
         self.q_norm, self.k_norm, self.mix = as_float(s.q_norm), as_float(s.k_norm), as_float(s.value_mix)
+        self.bias = None
+        if s.q_bias or s.k_bias or s.v_bias:
+            widths = (s.num_heads * s.dim, s.num_kv_heads * s.dim, self.v_dim)
+            self.bias = torch.cat([as_float(name) if name else torch.zeros(width, dtype=torch.float32, device=rt.device)
+                                   for name, width in zip((s.q_bias, s.k_bias, s.v_bias), widths)]).contiguous()
+        self.output_bias = as_float(s.o_bias)
         self.sink = None
         if s.sink_score is not None:
             self.sink = torch.full((s.num_heads,), float(s.sink_score), dtype=torch.float32, device=rt.device)
@@ -113,11 +122,13 @@ class NormedAttention(Mixer):
                           cos_sin=self.position.fusion_table(step.max_ctx) if self.position is not None else None,
                           rotated=s.rope.dims if s.rope is not None else 0,
                           interleaved=bool(s.rope is not None and s.rope.interleaved), mix=self.mix, first=first, keep=keep,
-                          write_kv=writes_cache)
+                          write_kv=writes_cache, bias=self.bias)
         ctx = rt.workspace.get("attn_ctx", (n, self.ctx_width), rt.dtype)
         attend_with_sink(step, rt, q, ctx, k_cache, v_cache, table, s.num_heads, s.num_kv_heads, self.key_width,
                          self.value_width, s.scale, sink=self.sink)
         ops.linear(ctx, self.w_o, x, _residual_mode(step), stats=_residual_stats(step))
+        if self.output_bias is not None and not self.leaves_output_bias:
+            ops.add_biased(x, None, self.output_bias, 1.0)
 
 
 register_mixer("normed_attention", NormedAttention)

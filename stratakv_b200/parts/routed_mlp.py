@@ -6,7 +6,7 @@ shared expert if the layer has one.
                                                  keep_groups best groups, a group scoring what its best expert does)
     y = sum over chosen e of s_e * route_scale * down_e act(up_e h)          (weights divided by their sum first if
                                                                                the spec says `renormalize`)
-      + sigmoid(shared.gate . h) * shared.down act(shared.up h)
+      + sigmoid(shared.gate . h) * shared.down act(shared.up h)      (or a gated unit, act(shared.unit_gate h) * (shared.up h))
 
 With ``spec.weigh_input`` the weights multiply the experts' inputs instead: ``y = sum over chosen e of
 expert_e(s_e * route_scale * h)``.
@@ -73,6 +73,8 @@ class RoutedMlp(FeedForward):
         if spec.shared is not None:
             wanted[spec.shared.up_weight] = TensorRequest((spec.shared.intermediate_size, spec.hidden_size))
             wanted[spec.shared.down_weight] = TensorRequest((spec.hidden_size, spec.shared.intermediate_size))
+            if getattr(spec.shared, "unit_gate_weight", None) is not None:
+                wanted[spec.shared.unit_gate_weight] = TensorRequest((spec.shared.intermediate_size, spec.hidden_size))
             if spec.shared.gate_weight is not None:
                 wanted[spec.shared.gate_weight] = TensorRequest((1, spec.hidden_size))
         return wanted
@@ -105,6 +107,10 @@ class RoutedMlp(FeedForward):
         if s.shared is not None:
             self.shared_up, self.shared_down = self._padded(rt.upload(tensors[s.shared.up_weight]),
                                                             rt.upload(tensors[s.shared.down_weight]), self.shared_padded)
+            unit_gate = getattr(s.shared, "unit_gate_weight", None)
+            self.shared_gated = unit_gate is not None
+            if self.shared_gated:
+                self.shared_up = pack_gate_up(rt.upload(tensors[unit_gate]), self.shared_up[:s.shared.intermediate_size])
             if s.shared.gate_weight is not None:
                 self.shared_gate = rt.upload(tensors[s.shared.gate_weight]).reshape(-1).contiguous()
 
@@ -143,7 +149,11 @@ class RoutedMlp(FeedForward):
         shared_out = None
         if self.shared_up is not None:
             z = get("ffn_hidden", (n, self.shared_padded), rt.dtype)
-            ops.linear(h, self.shared_up, z, _ops.MODE_ACT, s.activation)
+            if self.shared_gated:
+                ops.linear(h, self.shared_up, z, _ops.MODE_GATED, s.activation,
+                           activation_param=getattr(s, "activation_param", 0.0))
+            else:
+                ops.linear(h, self.shared_up, z, _ops.MODE_ACT, s.activation)
             shared_out = get("routed_shared", (n, s.hidden_size), torch.float32)
             ops.linear(z, self.shared_down, shared_out, _ops.MODE_STORE_F32)
         ops.combine_experts(results, place, None if self.weigh_input else weights, shared_out, share, x, add=not getattr(step, "store_branch", False))

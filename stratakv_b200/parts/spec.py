@@ -25,6 +25,8 @@ class NormSpec:
     # from one (``y = x / rms * (1 + w)``)
     weight_offset: float = 0.0
     groups: int = 1
+    # a factor on the weight, applied when it is loaded (a norm behind a sublayer whose result joins the stream with it)
+    weight_scale: float = 1.0
 
 
 @dataclass(frozen=True)
@@ -228,6 +230,8 @@ class NormedAttentionSpec:
     (``rope``), ``score = (q . k) scale``, and a softmax whose denominator also counts ``exp(sink_score)`` (one constant for
     all heads, with no key and no value; None: none).
 
+    ``q_bias`` / ``k_bias`` / ``v_bias`` are added to the projections first, ``o_bias`` to the result.
+
     Values may be shared along the layers: a layer that ``keeps_values`` leaves its values for the layers after it in the
     same step, and one with ``value_mix`` (a tensor name, one number m) has the values ``(1 - m) v + m kept`` and caches
     those."""
@@ -249,6 +253,10 @@ class NormedAttentionSpec:
     keeps_values: bool = False
     value_mix: Optional[str] = None
     kind: str = "normed_attention"
+    q_bias: Optional[str] = None     # tensor names
+    k_bias: Optional[str] = None
+    v_bias: Optional[str] = None
+    o_bias: Optional[str] = None
 
     @property
     def kernel_head_dim(self) -> int:
@@ -304,6 +312,94 @@ class Mamba2Spec:
 
 
 @dataclass(frozen=True)
+class ExpGateMemorySpec:
+    """A matrix memory with exponential gates (the mLSTM of the xLSTM family).  ``q = Wq h dim^-1/2``, ``k = Wk h`` (heads x
+    dim), ``v = Wv h`` (heads x vdim); per head ``i = cap tanh((Wi h + bi) / cap)``, ``f = log sigmoid(cap tanh((Wf h + bf) /
+    cap))``; with a running maximum m (0 at the start) ``m' = max(f + m, i)``, ``S' = exp(f + m - m') S + exp(i - m') k v^T``,
+    n likewise with k alone (both float32, zero at the start), ``o = S'^T q / (max(|n' . q|, exp(-m')) + denominator_eps)``;
+    every head of o over its root mean square, times ``norm``, times ``sigmoid(Wg h)``, then ``Wo``."""
+    hidden_size: int
+    num_heads: int
+    dim: int
+    vdim: int
+    gate_cap: float
+    denominator_eps: float
+    eps: float
+    q_weight: str                    # [heads * dim, hidden]
+    k_weight: str
+    v_weight: str                    # [heads * vdim, hidden]
+    input_weight: str                # [heads, hidden]
+    input_bias: str                  # [heads]
+    forget_weight: str
+    forget_bias: str
+    gate_weight: str                 # [heads * vdim, hidden]
+    norm: str                        # [heads * vdim]
+    o_weight: str                    # [hidden, heads * vdim]
+    kind: str = "exp_gate_memory"
+
+
+@dataclass(frozen=True)
+class GatedLinearAttentionSpec:
+    """Linear attention with a decay per token, head and key channel (GLA): ``q = Wq h dim^-1/2``, ``k = Wk h`` (heads x dim),
+    ``v = Wv h`` (heads x vdim), ``decay = sigmoid(Wa2 (Wa1 h) + ba)^(1 / tau)`` (heads x dim); per head ``S' = diag(decay) S +
+    k v^T`` (float32, zero at the start), ``o = S'^T q``; every head of o over its root mean square, times ``norm`` (one for
+    all heads), times ``silu(Wg h)``, then ``Wo``."""
+    hidden_size: int
+    num_heads: int
+    dim: int
+    vdim: int
+    tau: float
+    decay_rank: int
+    eps: float
+    q_weight: str                    # [heads * dim, hidden]
+    k_weight: str
+    v_weight: str                    # [heads * vdim, hidden]
+    gate_weight: str                 # [heads * vdim, hidden]
+    decay_down: str                  # Wa1, [rank, hidden]
+    decay_up: str                    # Wa2, [heads * dim, rank]
+    decay_bias: str                  # [heads * dim]
+    norm: str                        # [vdim]
+    o_weight: str                    # [hidden, heads * vdim]
+    kind: str = "gated_linear_attention"
+
+
+@dataclass(frozen=True)
+class GatedDeltaRuleSpec:
+    """The gated delta rule with a decay per token, head and key channel.  ``q, k = silu(conv(Wq h)), silu(conv(Wk h))``
+    (kv_heads x dim, shared by the heads of a group), ``v = silu(conv(Wv h))`` (heads x vdim), conv causal, per channel,
+    ``taps`` wide, without a bias; queries and keys of every head over ``sqrt(sum of squares + unit_eps)``, queries also times
+    ``dim^-1/2``; ``beta = sigmoid(Wb h)`` per head, ``decay = exp(-exp(A_log_head) softplus(Wa2 (Wa1 h) + dt_bias))``; per
+    head ``S <- diag(decay) S; S <- S + k (beta (v - S^T k))^T; o = S^T q`` (float32, zero at the start); every head of o over
+    its root mean square, times ``norm`` (one for all heads), times ``sigmoid(Wg2 (Wg1 h))``, then ``Wo``."""
+    hidden_size: int
+    num_heads: int
+    num_kv_heads: int
+    dim: int
+    vdim: int
+    taps: int
+    decay_rank: int
+    gate_rank: int
+    unit_eps: float
+    eps: float
+    q_weight: str                    # [kv_heads * dim, hidden]
+    k_weight: str
+    v_weight: str                    # [heads * vdim, hidden]
+    q_conv: str                      # [channels, taps], the last column weighs the current token
+    k_conv: str
+    v_conv: str
+    beta_weight: str                 # [heads, hidden]
+    a_log: str                       # [heads]
+    decay_down: str                  # Wa1, [decay_rank, hidden]
+    decay_up: str                    # Wa2, [heads * dim, decay_rank]
+    dt_bias: str                     # [heads * dim]
+    gate_down: str                   # Wg1, [gate_rank, hidden]
+    gate_up: str                     # Wg2, [heads * vdim, gate_rank]
+    norm: str                        # [vdim]
+    o_weight: str                    # [hidden, heads * vdim]
+    kind: str = "gated_delta_rule"
+
+
+@dataclass(frozen=True)
 class TimeMixSpec:
     """Time mixing with a matrix state per head and a decay per token and key channel (the RWKV family).  With h' the
     token before's input (zeros for the first), every projection s of r, k, v, g, w reads ``h + (h' - h) mu_s``;
@@ -340,6 +436,12 @@ class MixerPairSpec:
     left_scale: float = 1.0
     right_scale: float = 1.0
     kind: str = "mixer_pair"
+
+    @property
+    def kernel_head_dim(self) -> int:
+        """The head size whose compiled attention kernels serve one of the sides; 0: none names one."""
+        sizes = [getattr(side, "kernel_head_dim", None) or getattr(side, "head_dim", None) for side in (self.left, self.right)]
+        return next((size for size in sizes if size), 0)
 
 
 @dataclass(frozen=True)
@@ -411,11 +513,13 @@ class MlpSpec:
 
 @dataclass(frozen=True)
 class SharedExpertSpec:
-    """An expert every token uses; ``gate_weight`` ``[1, hidden]``: its result times ``sigmoid(gate_weight . h)``."""
+    """An expert every token uses; ``gate_weight`` ``[1, hidden]``: its result times ``sigmoid(gate_weight . h)``.
+    ``unit_gate_weight`` ``[intermediate, hidden]``: a gated unit, ``down(act(unit_gate h) * (up h))``."""
     intermediate_size: int
     up_weight: str
     down_weight: str
     gate_weight: Optional[str] = None
+    unit_gate_weight: Optional[str] = None
 
 
 @dataclass(frozen=True)
@@ -475,6 +579,8 @@ class LayerSpec:
     its two norms) may be ``None``.
     ``multi_stream``: the ``pre_norm`` block over several copies of the stream; the extras ``mixer_streams`` and
     ``ffn_streams`` (``StreamMixSpec``) say how each sublayer reads and writes them; ``ffn`` may be ``None``.
+    ``output_norm``: ``x += post1(mixer(x)); x += post2(ffn(x))``: the sublayers read the stream itself and only what they
+    give is normed (the extras ``mixer_post_norm`` and ``ffn_post_norm``); no norms in front, ``ffn`` may be ``None``.
     ``parallel_pair``: ``x += mixer(norm1(x)) + ffn(norm2(x))``, both norms of the same x, then ``token_input`` if the
     layer has one; ``ffn`` (with its norm) may be ``None``.
 
@@ -551,12 +657,13 @@ class SummedEmbeddingSpec:
 @dataclass(frozen=True)
 class HeadSpec:
     """Final norm on the wanted rows, then ``logits = y . W^T`` (``src/generation/generator.cpp:773-774``)
-    times ``logit_scale``.  ``weight`` may be the embedding table's name (tied)."""
+    times ``logit_scale``, then ``softcap * tanh(logits / softcap)`` if softcap is not 0.  ``weight`` may be the embedding table's name (tied)."""
     vocab_size: int
     hidden_size: int
     weight: str
     kind: str = "linear_head"
     logit_scale: float = 1.0
+    softcap: float = 0.0
 
 
 @dataclass(frozen=True)
