@@ -7,6 +7,8 @@
     python bench.py --design fidolix [--layers 8]       (the Fidolix decoder beside Llama and beside the Kedelorn decoder)
     python bench.py --design tobozen [--layers 9]       (the Tobozen decoder beside Llama and beside the nearest layers of the
                                                          Kedelorn and Fidolix decoders: mixed layers, and each mixer alone)
+    python bench.py --design vekanex [--layers 9]       (the Vekanex decoder beside Llama and beside the nearest layers of the
+                                                         Tobozen and Fidolix decoders: mixed layers, and each mixer alone)
     python bench.py --design kedelorn [--layers 8]      (the Kedelorn decoder beside Llama and beside Povusun's latent and
                                                          recurrent layers: mixed layers, and each of its two mixers alone)
 
@@ -448,10 +450,56 @@ def tobozen_config(size, layers, vocab, kinds):
                                     "norm": {"eps": 1e-5, "groups": 2}, "layers": made})
 
 
-def tobozen_arm(args) -> int:
-    """Prefill and decode of the Tobozen decoder beside the Llama decoder and beside the framework's nearest layers
-    (Kedelorn's retention, a matrix state with a decay per head; Fidolix's attention layer, with the same experts) at equal
-    layer sizes, random weights: a model that alternates its three kinds of layer, and one of each kind alone."""
+def tobozen_models(size, layers, vocab):
+    """Tobozen's models, one that alternates its three kinds of layer and one of each kind alone, behind the framework's
+    nearest layers: Kedelorn's retention (a matrix state with a decay per head) and Fidolix's attention layer, with the same
+    experts."""
+    return {"kedelorn_retention_only": kedelorn_config(size, layers, vocab, ("retention",)),
+            "fidolix_attention_only": fidolix_config(size, layers, vocab, ("attention",)),
+            "tobozen": tobozen_config(size, layers, vocab, ("attention", "mamba2", "lightning")),
+            "tobozen_attention_only": tobozen_config(size, layers, vocab, ("attention",)),
+            "tobozen_mamba2_only": tobozen_config(size, layers, vocab, ("mamba2",)),
+            "tobozen_lightning_only": tobozen_config(size, layers, vocab, ("lightning",))}
+
+
+def vekanex_config(size, layers, vocab, kinds):
+    """A Vekanex configuration at a size of DESIGN_SIZES whose layer i has the mixer ``kinds[i % len(kinds)]``.  The memories
+    with exponential gates, the gated linear attention (decays of rank 16) and the right side of a parallel layer (four taps,
+    decays and gate of the head size's rank) have Llama's heads with keys and values of the head size; its left side has
+    Llama's heads, key heads and head size, the whole head rotated.  Every layer has eight experts of which two are chosen,
+    each a quarter as wide as Llama's feed-forward, and a shared one half as wide, so that a token passes through as many
+    feed-forward weights as in Llama.  No layer uses another's weights (the arms have equal numbers of layers)."""
+    from stratakv_b200.config import VekanexConfig
+    d, heads = size["head_dim"], size["heads"]
+    mlp = {"kind": "moe", "expert": {"ff": size["llama_ff"] // 4 // 64 * 64}, "router": {"experts": 8, "top": 2},
+           "shared": {"ff": size["llama_ff"] // 2 // 64 * 64}}
+    mixers = {
+        "mlstm": {"heads": heads, "dim": d, "vdim": d, "gate_cap": 15.0},
+        "gla": {"heads": heads, "dim": d, "vdim": d, "tau": 16.0, "rank": 16},
+        "parallel": {"left": {"heads": heads, "kv_heads": size["kv_heads"], "dim": d, "vdim": d, "scale": d ** -0.5,
+                              "rot": {"dims": d, "base": 10000.0}},
+                     "right": {"heads": heads, "kv_heads": heads, "dim": d, "vdim": d, "conv": 4, "decay_rank": d, "gate_rank": d},
+                     "left_scale": 0.8, "right_scale": 0.6}}
+    made = [{"type": kinds[i % len(kinds)], "mixer": mixers[kinds[i % len(kinds)]], "mlp": mlp} for i in range(layers)]
+    return VekanexConfig.from_dict({"architecture": "Vekanex", "vocab": vocab, "width": size["hidden"], "norm": {"eps": 1e-5},
+                                    "residual_mult": 0.7, "logit_softcap": 30.0, "layers": made})
+
+
+def vekanex_models(size, layers, vocab):
+    """Vekanex's models behind the framework's nearest layers: Tobozen's Lightning (a matrix state with a decay per head,
+    experts of the same kind), its attention (norms over all heads, rotation) and Fidolix's parallel layer (attention beside a
+    matrix state with a decay per key channel)."""
+    return {"tobozen_lightning_only": tobozen_config(size, layers, vocab, ("lightning",)),
+            "fidolix_parallel_only": fidolix_config(size, layers, vocab, ("parallel",), 1 << 20),
+            "vekanex": vekanex_config(size, layers, vocab, ("gla", "mlstm", "parallel")),
+            "vekanex_mlstm_only": vekanex_config(size, layers, vocab, ("mlstm",)),
+            "vekanex_gla_only": vekanex_config(size, layers, vocab, ("gla",)),
+            "vekanex_parallel_only": vekanex_config(size, layers, vocab, ("parallel",))}
+
+
+def nearest_arm(args, design, beside, models_of) -> int:
+    """Prefill and decode of a design's models beside the Llama decoder and beside the framework's nearest layers at equal
+    layer sizes, random weights."""
     import gc
     import torch
     from stratakv_b200.config import LlamaConfig
@@ -470,13 +518,7 @@ def tobozen_arm(args) -> int:
         configs = {"llama": LlamaConfig.from_dict(dict(
             TINYLLAMA, hidden_size=size["hidden"], intermediate_size=size["llama_ff"], num_hidden_layers=layers,
             num_attention_heads=size["heads"], num_key_value_heads=size["kv_heads"], head_dim=size["head_dim"],
-            vocab_size=vocab, max_position_embeddings=context + 64)),
-            "kedelorn_retention_only": kedelorn_config(size, layers, vocab, ("retention",)),
-            "fidolix_attention_only": fidolix_config(size, layers, vocab, ("attention",)),
-            "tobozen": tobozen_config(size, layers, vocab, ("attention", "mamba2", "lightning")),
-            "tobozen_attention_only": tobozen_config(size, layers, vocab, ("attention",)),
-            "tobozen_mamba2_only": tobozen_config(size, layers, vocab, ("mamba2",)),
-            "tobozen_lightning_only": tobozen_config(size, layers, vocab, ("lightning",))}
+            vocab_size=vocab, max_position_embeddings=context + 64)), **models_of(size, layers, vocab)}
         only = [label for label in args.arms.split(",") if label] if args.arms else list(configs)
         row = {}
         for label in only:
@@ -502,7 +544,7 @@ def tobozen_arm(args) -> int:
                 row[label]["decode_ratio"] = row[label]["decode_tokens_per_s"] / row["llama"]["decode_tokens_per_s"]
         sizes[name] = row
     clocks = sampler.stop()
-    print(json.dumps({"design": "Tobozen", "beside": ["LlamaForCausalLM", "Kedelorn", "Fidolix"], "layers": layers, "vocab": vocab,
+    print(json.dumps({"design": design, "beside": beside, "layers": layers, "vocab": vocab,
                       "prefill_tokens": PREFILL_TOKENS, "decode_batch": batch, "context": context, "dtype": "bf16",
                       "steps": steps, "warmup": warmup,
                       "data": "synthetic: random N(0,0.02) weights, uniform random token ids", "peaks": peak,
@@ -513,7 +555,9 @@ def tobozen_arm(args) -> int:
 def design_arm(args) -> int:
     """Prefill and decode of the Zepavik decoder and of the Llama decoder at equal layer sizes (random weights)."""
     if args.design == "tobozen":
-        return tobozen_arm(args)
+        return nearest_arm(args, "Tobozen", ["LlamaForCausalLM", "Kedelorn", "Fidolix"], tobozen_models)
+    if args.design == "vekanex":
+        return nearest_arm(args, "Vekanex", ["LlamaForCausalLM", "Tobozen", "Fidolix"], vekanex_models)
     if args.design == "fidolix":
         return fidolix_arm(args)
     if args.design == "povusun":
@@ -869,10 +913,10 @@ def main() -> int:
     parser.add_argument("--impl", default="ours", choices=["ours", "reference"])
     parser.add_argument("--skip-points", action="store_true", help="leave out batch 1 and 64 and the prefill")
     parser.add_argument("--context", type=int, default=CONTEXT, help="context at which the timed decode steps end")
-    parser.add_argument("--design", choices=["zepavik", "povusun", "kedelorn", "fidolix", "tobozen"],
+    parser.add_argument("--design", choices=["zepavik", "povusun", "kedelorn", "fidolix", "tobozen", "vekanex"],
                         help="measure this design beside the Llama decoder at equal layer sizes instead of the step benchmark")
     parser.add_argument("--sizes", default="", help="with --design: names of DESIGN_SIZES, with commas (default: all)")
-    parser.add_argument("--arms", default="", help="with --design kedelorn, fidolix or tobozen: which models to time, with commas (default: all)")
+    parser.add_argument("--arms", default="", help="with --design kedelorn, fidolix, tobozen or vekanex: which models to time, with commas (default: all)")
     parser.add_argument("--window", type=int, default=0, help="with --design: the design's window (default: the whole context)")
     parser.add_argument("--workload", choices=sorted(WORKLOADS),
                         help="a whole generation workload through Engine.generate instead of the step benchmark")

@@ -95,6 +95,7 @@ route_tokens_kernel(const T* __restrict__ h, const T* __restrict__ router, const
         float total = 0.0f;
         for (int e = lane; e < experts; e += 32) {
             const float w = expf(score[e] - top_logit);
+            choice[e] = score[e];                     // (logits order experts whose shares are too small to tell apart)
             score[e] = w;
             total += w;
         }
@@ -103,7 +104,8 @@ route_tokens_kernel(const T* __restrict__ h, const T* __restrict__ router, const
         for (int e = lane; e < experts; e += 32) {
             const float s = score[e] / total;
             score[e] = s;
-            choice[e] = correction ? s + correction[e] : s;
+            if (correction) choice[e] = s + correction[e];
+            else if (groups > 1) choice[e] = s;
         }
         __syncwarp();
     }

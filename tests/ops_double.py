@@ -195,7 +195,8 @@ class DoubleKernels:
         self.calls.append("rmsnorm_add")
         x.add_(y / torch.sqrt((y * y).mean(dim=-1, keepdim=True) + eps) * gamma)
         if next_out is not None:
-            next_out.copy_((x / torch.sqrt((x * x).mean(dim=-1, keepdim=True) + next_eps) * next_gamma).to(next_out.dtype))
+            normed = x if next_gamma is None else x / torch.sqrt((x * x).mean(dim=-1, keepdim=True) + next_eps) * next_gamma
+            next_out.copy_(normed.to(next_out.dtype))
 
     def token_side(self, x, ids, table, offset, dim, gate_w, proj_t, norm_w, eps, next_gamma=None, next_eps=0.0,
                    next_out=None, branch=None, post_gamma=None, post_eps=0.0):
@@ -423,6 +424,14 @@ class DoubleKernels:
         self.calls.append("add_scaled")
         out.add_(other * factor)
 
+    def add_biased(self, out, other, bias, factor):
+        self.calls.append("add_biased")
+        out.add_(((other if other is not None else 0.0) + bias) * factor)
+
+    def softcap_inplace(self, x, cap):
+        self.calls.append("softcap_inplace")
+        x.copy_(cap * torch.tanh(x / cap))
+
     def projection_norm(self, rows, eps, segments):
         self.calls.append("projection_norm")
         for offset, width, bias, weight in segments:
@@ -536,9 +545,11 @@ class DoubleKernels:
 
     def normed_rotary(self, rows, q_out, k_cache, v_cache, positions, token_seq, block_table, num_heads, num_kv_heads, dim,
                       vdim, block_size, eps=0.0, q_weight=None, k_weight=None, cos_sin=None, rotated=0, interleaved=False,
-                      mix=None, first=None, keep=None, write_kv=True):
+                      mix=None, first=None, keep=None, write_kv=True, bias=None):
         self.calls.append("normed_rotary")
         n = rows.shape[0]
+        if bias is not None:
+            rows = rows[:, :bias.numel()] + bias
         a, b, c = num_heads * dim, num_kv_heads * dim, num_kv_heads * vdim
 
         def turned(x, weight, heads):
@@ -575,11 +586,12 @@ class DoubleKernels:
                 row.zero_()
                 row[:, :value.shape[-1]] = value.to(cache.dtype)
 
-    def linear_state_scratch(self, n_seqs, max_q_len, heads, dim, vdim):
+    def linear_state_scratch(self, n_seqs, max_q_len, heads, dim, vdim, with_floor=False):
         return 0
 
     def linear_state(self, rows, q_at, k_at, v_at, out, state, step_meta, heads, groups, dim, vdim, max_q_len, decay=None,
-                     log_decay=None, key_scale=None, skip=None, silu=False, scratch=None, state_offset=0):
+                     log_decay=None, key_scale=None, skip=None, silu=False, scratch=None, state_offset=0, out_scale=1.0,
+                     floor=None, floor_eps=0.0):
         self.calls.append("linear_state")
         positions, token_seq, cu_q, slot_ids = step_meta
         n = rows.shape[0]
@@ -592,17 +604,24 @@ class DoubleKernels:
             k = k * key_scale[:, :, None]
         d = decay.expand(n, heads) if decay is not None else torch.exp(log_decay)
         size = heads * dim * vdim
+        half = size + (heads * dim if floor is not None else 0)
         for s in range(slot_ids.numel()):
             first, last = int(cu_q[s]), int(cu_q[s + 1]) - 1
             row = state[int(slot_ids[s])][state_offset:]
             p_first = int(positions[first])
-            S = (row[((p_first - 1) & 1) * size:][:size].clone().view(heads, dim, vdim) if p_first > 0
-                 else torch.zeros(heads, dim, vdim))
+            before = row[((p_first - 1) & 1) * half:][:half].clone() if p_first > 0 else torch.zeros(half)
+            S, sums = before[:size].view(heads, dim, vdim), before[size:].view(-1, dim)
             for t in range(first, last + 1):
                 S = d[t][:, None, None] * S + k[t][:, :, None] * v[t][:, None, :]
-                o = torch.einsum("hnp,hn->hp", S, q[t])
+                o = torch.einsum("hnp,hn->hp", S, q[t]) * out_scale
+                if floor is not None:
+                    sums = d[t][:, None] * sums + k[t]
+                    dot = (sums * q[t]).sum(dim=-1).abs() * out_scale
+                    o = o / (torch.maximum(dot, floor[t]) + floor_eps)[:, None]
                 out[t] = (o + skip[:, None] * v[t] if skip is not None else o).reshape(-1)
-            row[((p_first + last - first) & 1) * size:][:size] = S.reshape(size)
+            after = row[((p_first + last - first) & 1) * half:]
+            after[:size] = S.reshape(-1)
+            after[size:half] = sums.reshape(-1)
 
     def conv_silu(self, rows, conv_w, conv_b, out, step_meta, state, ring_offset=0):
         self.calls.append("conv_silu")
@@ -611,7 +630,7 @@ class DoubleKernels:
         for t in range(rows.shape[0]):
             seq, p = int(token_seq[t]), int(positions[t])
             first = int(cu_q[seq])
-            y = conv_b.clone()
+            y = conv_b.clone() if conv_b is not None else torch.zeros(channels)
             for j in range(taps):
                 back = taps - 1 - j
                 if p - back < 0:
@@ -642,15 +661,99 @@ class DoubleKernels:
                           log_decay=log_decay, key_scale=dt, skip=skip, state_offset=state_offset)
         self.short_conv_remember(rows, None, channels, taps, n, step_meta, state, ring_offset)
 
-    def gated_norm(self, y, gate, gate_stride, weight, groups, eps, gate_first, out):
+    def gated_norm(self, y, gate, gate_stride, weight, groups, eps, mode, out):
         self.calls.append("gated_norm")
         n, width = y.shape
         g = gate[:, :width]
-        x = y * ACTIVATIONS["silu"](g) if gate_first else y
+        x = y * ACTIVATIONS["silu"](g) if mode == 1 else y
         parts = x.view(n, groups, -1)
         x = (parts / torch.sqrt((parts * parts).mean(dim=-1, keepdim=True) + eps)).reshape(n, width) * weight
         out.zero_()
-        out[:, :width] = (x if gate_first else x * torch.sigmoid(g)).to(out.dtype)
+        out[:, :width] = (x * {0: torch.sigmoid(g), 1: 1.0, 2: ACTIVATIONS["silu"](g)}[mode]).to(out.dtype)
+
+    def exp_gates(self, rows, input_at, forget_at, input_bias, forget_bias, cap, log_decay, key_scale, floor, step_meta, state,
+                  m_offset=0):
+        self.calls.append("exp_gates")
+        positions, token_seq, cu_q, slot_ids = step_meta
+        heads = input_bias.numel()
+        i = cap * torch.tanh((rows[:, input_at:input_at + heads] + input_bias) / cap)
+        f = torch.nn.functional.logsigmoid(cap * torch.tanh((rows[:, forget_at:forget_at + heads] + forget_bias) / cap))
+        for s in range(slot_ids.numel()):
+            first, end = int(cu_q[s]), int(cu_q[s + 1])
+            kept = state[int(slot_ids[s])][m_offset:m_offset + 2 * heads].view(2, heads)
+            p = int(positions[first])
+            m = kept[(p - 1) & 1].clone() if p > 0 else torch.zeros(heads)
+            for t in range(first, end):
+                top = torch.maximum(f[t] + m, i[t])
+                log_decay[t], key_scale[t], floor[t] = f[t] + m - top, torch.exp(i[t] - top), torch.exp(-top)
+                m = top
+            kept[(p + end - first - 1) & 1] = m
+
+    def low_rank(self, rows, at, wt, out, bias=None, mode=0, factor=1.0, rate=None):
+        self.calls.append("low_rank")
+        z = rows[:, at:at + wt.shape[0]] @ wt.float()
+        if bias is not None:
+            z = z + bias
+        if mode == 1:
+            z = torch.nn.functional.logsigmoid(z) * factor
+        elif mode == 2:
+            z = -torch.nn.functional.softplus(z) * rate.repeat_interleave(z.shape[1] // rate.numel())
+        out.copy_(z)
+
+    def channel_state_scratch(self, n_tokens, n_seqs, max_q_len, heads, dim, vdim, delta):
+        return 4
+
+    def channel_state(self, rows, q_at, k_at, v_at, log_decay, out, state, step_meta, heads, groups, dim, vdim, max_q_len, scratch,
+                      q_scale=1.0, beta_rows=None, beta_at=0, unit_eps=None, state_offset=0):
+        self.calls.append("channel_state")
+        positions, token_seq, cu_q, slot_ids = step_meta
+        n = rows.shape[0]
+        unit = (lambda x: x) if unit_eps is None else (lambda x: x / torch.sqrt((x * x).sum(dim=-1, keepdim=True) + unit_eps))
+        spread = lambda at: unit(rows[:, at:at + groups * dim].view(n, groups, dim)).repeat_interleave(heads // groups, dim=1)
+        q, k, v = spread(q_at) * q_scale, spread(k_at), rows[:, v_at:v_at + heads * vdim].view(n, heads, vdim)
+        d = torch.exp(log_decay).view(n, heads, dim)
+        size = heads * dim * vdim
+        for s in range(slot_ids.numel()):
+            first, end = int(cu_q[s]), int(cu_q[s + 1])
+            row = state[int(slot_ids[s])][state_offset:]
+            p = int(positions[first])
+            S = row[((p - 1) & 1) * size:][:size].clone().view(heads, dim, vdim) if p > 0 else torch.zeros(heads, dim, vdim)
+            for t in range(first, end):
+                S = d[t][:, :, None] * S
+                u = v[t]
+                if beta_rows is not None:
+                    u = torch.sigmoid(beta_rows[t, beta_at:beta_at + heads])[:, None] * (u - torch.einsum("hnp,hn->hp", S, k[t]))
+                S = S + k[t][:, :, None] * u[:, None, :]
+                out[t] = torch.einsum("hnp,hn->hp", S, q[t]).reshape(-1)
+            row[((p + end - first - 1) & 1) * size:][:size] = S.reshape(-1)
+
+    def matrix_step(self, kind, rows, q_at, k_at, v_at, out, state, step_meta, heads, groups, dim, vdim, norm, eps, gate_at,
+                    q_scale=1.0, unit_eps=None, conv_w=None, ring_offset=0, decay_at=0, decay_wt=None, decay_bias=None, decay_mode=1,
+                    decay_factor=1.0, decay_rate=None, beta_at=0, input_at=0, forget_at=0, input_bias=None, forget_bias=None,
+                    cap=1.0, denominator_eps=0.0, gate_wt=None, gate_silu=False, state_offset=0):
+        self.calls.append("matrix_step")
+        n, hp = rows.shape[0], heads * vdim
+        y = torch.zeros(n, hp)
+        if kind == 2:
+            decay, scale, floor = torch.zeros(n, heads), torch.zeros(n, heads), torch.zeros(n, heads)
+            self.exp_gates(rows, input_at, forget_at, input_bias, forget_bias, cap, decay, scale, floor, step_meta, state,
+                           state_offset + 2 * heads * dim * (vdim + 1))
+            self.linear_state(rows, q_at, k_at, v_at, y, state, step_meta, heads, groups, dim, vdim, 1, log_decay=decay,
+                              key_scale=scale, state_offset=state_offset, out_scale=q_scale, floor=floor, floor_eps=denominator_eps)
+        else:
+            log_decay = torch.zeros(n, heads * dim)
+            self.low_rank(rows, decay_at, decay_wt, log_decay, decay_bias, decay_mode, decay_factor, decay_rate)
+            inputs, beta = rows, None
+            if kind == 1:
+                inputs, beta = torch.zeros(n, conv_w.shape[0]), rows
+                self.conv_silu(rows, conv_w, None, inputs, step_meta, state, ring_offset)
+                self.short_conv_remember(rows, None, conv_w.shape[0], conv_w.shape[1], n, step_meta, state, ring_offset)
+            self.channel_state(inputs, q_at, k_at, v_at, log_decay, y, state, step_meta, heads, groups, dim, vdim, 1, None,
+                               q_scale, beta, beta_at, unit_eps, state_offset)
+        gate = rows[:, gate_at:gate_at + hp]
+        if gate_wt is not None:
+            gate = rows[:, gate_at:gate_at + gate_wt.shape[0]] @ gate_wt.float()
+        self.gated_norm(y, gate, 0, norm, heads, eps, 2 if gate_silu else 0, out)
 
     def scale_inplace(self, x, factor):
         x.mul_(factor)
