@@ -30,7 +30,8 @@
 
 namespace skv {
 
-constexpr int CS_OUT_THREADS = 128;
+constexpr int CS_PREPARE_THREADS = 128, CS_OUT_THREADS = 256;
+constexpr float CS_LOG2E = 1.4426950408889634f;        // (inside a chunk decays are kept as powers of two)
 
 struct ChannelShape {
     int heads, groups, dim, vdim;
@@ -70,8 +71,24 @@ __device__ __forceinline__ float low_rank_end(const LowRankEnd& end, float z, in
     return z;
 }
 
-// A block takes TOK tokens and 256 channels, a thread a channel: a weight that is read serves all of the block's tokens.
-template <typename T, int TOK>
+// A block takes TOK tokens and 256 EACH channels, a thread EACH neighbouring channels: a weight that is read serves all of the
+// block's tokens, and a token's number all of the thread's channels.
+template <int EACH>
+__device__ __forceinline__ void low_rank_weights(const float* p, float (&w)[EACH]) {
+#pragma unroll
+    for (int e = 0; e < EACH; ++e) w[e] = p[e];
+}
+template <int EACH>
+__device__ __forceinline__ void low_rank_weights(const __nv_bfloat16* p, float (&w)[EACH]) {
+    if (EACH == 2) {
+        const float2 pair = __bfloat1622float2(*(const __nv_bfloat162*)p);
+        w[0] = pair.x; w[EACH - 1] = pair.y;
+    } else {
+        w[0] = __bfloat162float(p[0]);
+    }
+}
+
+template <typename T, int TOK, int EACH>
 __global__ void __launch_bounds__(256)
 low_rank_kernel(const float* __restrict__ x, int x_stride, int rank, const T* __restrict__ wt, const LowRankEnd end,
                 float* __restrict__ out, int n_tokens, int channels) {
@@ -84,45 +101,64 @@ low_rank_kernel(const float* __restrict__ x, int x_stride, int rank, const T* __
         cs_smem[j * TOK + tok] = tok < count ? x[(size_t)(t0 + tok) * x_stride + j] : 0.0f;
     }
     __syncthreads();
-    const int c = blockIdx.y * 256 + threadIdx.x;
+    const int c = (blockIdx.y * 256 + threadIdx.x) * EACH;
     if (c >= channels) return;
-    float z[TOK];
-    const float bias = end.bias ? end.bias[c] : 0.0f;
+    float z[TOK][EACH];
 #pragma unroll
-    for (int tok = 0; tok < TOK; ++tok) z[tok] = bias;
-#pragma unroll 8
+    for (int e = 0; e < EACH; ++e) {
+        const float bias = end.bias ? end.bias[c + e] : 0.0f;
+#pragma unroll
+        for (int tok = 0; tok < TOK; ++tok) z[tok][e] = bias;
+    }
+#pragma unroll 4
     for (int j = 0; j < rank; ++j) {
-        const float w = to_float(wt[(size_t)j * channels + c]);
+        float w[EACH];
+        low_rank_weights<EACH>(wt + (size_t)j * channels + c, w);
 #pragma unroll
         for (int tok = 0; tok < TOK; tok += 4) {
             const float4 v = *(const float4*)(cs_smem + j * TOK + tok);
-            z[tok] = fmaf(w, v.x, z[tok]); z[tok + 1] = fmaf(w, v.y, z[tok + 1]);
-            z[tok + 2] = fmaf(w, v.z, z[tok + 2]); z[tok + 3] = fmaf(w, v.w, z[tok + 3]);
+#pragma unroll
+            for (int e = 0; e < EACH; ++e) {
+                z[tok][e] = fmaf(w[e], v.x, z[tok][e]); z[tok + 1][e] = fmaf(w[e], v.y, z[tok + 1][e]);
+                z[tok + 2][e] = fmaf(w[e], v.z, z[tok + 2][e]); z[tok + 3][e] = fmaf(w[e], v.w, z[tok + 3][e]);
+            }
         }
     }
 #pragma unroll
-    for (int tok = 0; tok < TOK; ++tok)
-        if (tok < count) out[(size_t)(t0 + tok) * channels + c] = low_rank_end(end, z[tok], c);
+    for (int tok = 0; tok < TOK; ++tok) {
+        if (tok >= count) continue;
+        float* to = out + (size_t)(t0 + tok) * channels + c;
+        if (EACH == 2) *(float2*)to = make_float2(low_rank_end(end, z[tok][0], c), low_rank_end(end, z[tok][EACH - 1], c + EACH - 1));
+        else to[0] = low_rank_end(end, z[tok][0], c);
+    }
 }
 
 // ---- chunks: what the three kernels share ------------------------------------------------------------------------
 __device__ __forceinline__ int cs_pad(int n) { return (n + 3) & ~3; }
 
+// Where a thread stands over rows of `width` items: its item of a row, its first row, and the rows between its turns (threads
+// past the last whole row have none).  Made once: divisions inside the loops would cost more than what the loops do.
+struct RowPlace { int row, item, rows, lanes; };
+template <int THREADS>
+__device__ __forceinline__ RowPlace row_place(int width) {
+    const int lanes = min(width, THREADS), rows = THREADS / lanes, row = threadIdx.x / lanes;
+    return {row < rows ? row : 1 << 20, (int)threadIdx.x - row * lanes, rows, lanes};
+}
+
 // to[t][n] (rows ld apart) = scale * from[t * stride + n], zero beyond L tokens and N numbers.
-template <int CH, int THREADS>
-__device__ __forceinline__ void load_chunk(float* to, int ld, const float* __restrict__ from, size_t stride, int L, int N, int n_pad) {
+template <int CH>
+__device__ __forceinline__ void load_chunk(float* to, int ld, const float* __restrict__ from, size_t stride, int L, int N, int n_pad,
+                                           const RowPlace& one, const RowPlace& four, float scale = 1.0f) {
     if (((stride | (size_t)N) & 3) == 0 && ((uintptr_t)from & 15) == 0) {
-        const int quads = n_pad >> 2;
+        for (int n = four.item * 4; n < n_pad; n += 4 * four.lanes)
 #pragma unroll 4
-        for (int idx = threadIdx.x; idx < CH * quads; idx += THREADS) {
-            const int t = idx / quads, n = (idx - t * quads) * 4;
-            *(float4*)(to + t * ld + n) = t < L ? *(const float4*)(from + t * stride + n) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-        }
+            for (int t = four.row; t < CH; t += four.rows) {
+                const float4 x = t < L ? *(const float4*)(from + t * stride + n) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+                *(float4*)(to + t * ld + n) = make_float4(x.x * scale, x.y * scale, x.z * scale, x.w * scale);
+            }
     } else {
-        for (int idx = threadIdx.x; idx < CH * n_pad; idx += THREADS) {
-            const int t = idx / n_pad, n = idx - t * n_pad;
-            to[t * ld + n] = t < L && n < N ? from[t * stride + n] : 0.0f;
-        }
+        for (int n = one.item; n < n_pad; n += one.lanes)
+            for (int t = one.row; t < CH; t += one.rows) to[t * ld + n] = t < L && n < N ? from[t * stride + n] * scale : 0.0f;
     }
 }
 
@@ -142,29 +178,32 @@ __device__ __forceinline__ void unit_rows(float* rows, int ld, int n_pad, float 
     }
 }
 
-// One level: scaled[t] of a right half is right[t] * exp(sum from the middle to t), of a left half left[t] * exp(sum behind t).
-template <int CH, int THREADS, int HALF>
-__device__ __forceinline__ void scale_level(float* scaled, const float* right, const float* left, const float* l, int ld, int n_pad) {
+// One level: scaled[t] of a right half is right[t] * 2^(sum from the middle to t), of a left half left[t] * 2^(sum behind t); l
+// holds the logarithms of the decays to base two.
+template <int CH, int HALF>
+__device__ __forceinline__ void scale_level(float* scaled, const float* right, const float* left, const float* l, int ld, int n_pad,
+                                            const RowPlace& one) {
     constexpr int SEGMENTS = CH / HALF;
-    for (int task = threadIdx.x; task < SEGMENTS * n_pad; task += THREADS) {
-        const int segment = task / n_pad, n = task - segment * n_pad, t0 = segment * HALF;
-        float sum = 0.0f;
-        if (segment & 1) {
-#pragma unroll
-            for (int t = 0; t < HALF; ++t) {
-                const int at = (t0 + t) * ld + n;
-                sum += l[at];
-                scaled[at] = right[at] * expf(sum);
-            }
-        } else {
-#pragma unroll
-            for (int t = HALF - 1; t >= 0; --t) {
-                const int at = (t0 + t) * ld + n;
-                scaled[at] = left[at] * expf(sum);
-                sum += l[at];
+    for (int n = one.item; n < n_pad; n += one.lanes)
+        for (int segment = one.row; segment < SEGMENTS; segment += one.rows) {
+            const int from = segment * HALF * ld + n;
+            float sum = 0.0f;
+            if (segment & 1) {
+#pragma unroll 8
+                for (int t = 0; t < HALF; ++t) {
+                    const int at = from + t * ld;
+                    sum += l[at];
+                    scaled[at] = right[at] * exp2f(sum);
+                }
+            } else {
+#pragma unroll 8
+                for (int t = HALF - 1; t >= 0; --t) {
+                    const int at = from + t * ld;
+                    scaled[at] = left[at] * exp2f(sum);
+                    sum += l[at];
+                }
             }
         }
-    }
 }
 
 __device__ __forceinline__ float cs_dot4(const float4 a, const float4 b, float acc) {
@@ -206,8 +245,9 @@ __device__ __forceinline__ void level_products(float* w, const float* scaled, in
 }
 
 template <int CH, int THREADS, int HALF>
-__device__ __forceinline__ void one_level(float* w, float* scaled, const float* right, const float* left, const float* l, int ld, int n_pad) {
-    scale_level<CH, THREADS, HALF>(scaled, right, left, l, ld, n_pad);
+__device__ __forceinline__ void one_level(float* w, float* scaled, const float* right, const float* left, const float* l, int ld, int n_pad,
+                                          const RowPlace& one) {
+    scale_level<CH, HALF>(scaled, right, left, l, ld, n_pad, one);
     __syncthreads();
     level_products<CH, THREADS, HALF>(w, scaled, ld, n_pad);
     __syncthreads();
@@ -215,29 +255,30 @@ __device__ __forceinline__ void one_level(float* w, float* scaled, const float* 
 
 // w[i][j] (rows CH + 4 apart) = sum_n right[i][n] left[j][n] E(j, i)[n] for j < i.  Tokens past the chunk's last hold zeros.
 template <int CH, int THREADS>
-__device__ __forceinline__ void decayed_products(float* w, float* scaled, const float* right, const float* left, const float* l, int ld, int n_pad) {
-    if constexpr (CH >= 32) one_level<CH, THREADS, 16>(w, scaled, right, left, l, ld, n_pad);
-    one_level<CH, THREADS, 8>(w, scaled, right, left, l, ld, n_pad);
-    one_level<CH, THREADS, 4>(w, scaled, right, left, l, ld, n_pad);
-    one_level<CH, THREADS, 2>(w, scaled, right, left, l, ld, n_pad);
-    one_level<CH, THREADS, 1>(w, scaled, right, left, l, ld, n_pad);
+__device__ __forceinline__ void decayed_products(float* w, float* scaled, const float* right, const float* left, const float* l, int ld,
+                                                 int n_pad, const RowPlace& one) {
+    if constexpr (CH >= 32) one_level<CH, THREADS, 16>(w, scaled, right, left, l, ld, n_pad, one);
+    one_level<CH, THREADS, 8>(w, scaled, right, left, l, ld, n_pad, one);
+    one_level<CH, THREADS, 4>(w, scaled, right, left, l, ld, n_pad, one);
+    one_level<CH, THREADS, 2>(w, scaled, right, left, l, ld, n_pad, one);
+    one_level<CH, THREADS, 1>(w, scaled, right, left, l, ld, n_pad, one);
 }
 
-// scaled[t] = x[t] * exp(l_0 + .. + l_t)
-template <int CH, int THREADS>
-__device__ __forceinline__ void scale_from_start(float* scaled, const float* x, const float* l, int ld, int n_pad) {
+// scaled[t] = x[t] * 2^(l_0 + .. + l_t)
+template <int CH>
+__device__ __forceinline__ void scale_from_start(float* scaled, const float* x, const float* l, int ld, int n_pad, const RowPlace& one) {
     constexpr int SEGMENT = CH / 4;
-    for (int task = threadIdx.x; task < 4 * n_pad; task += THREADS) {
-        const int segment = task / n_pad, n = task - segment * n_pad, t0 = segment * SEGMENT;
-        float sum = 0.0f;
-        for (int t = 0; t < t0; ++t) sum += l[t * ld + n];
+    for (int n = one.item; n < n_pad; n += one.lanes)
+        for (int segment = one.row; segment < 4; segment += one.rows) {
+            float sum = 0.0f;
+            for (int t = 0; t < segment * SEGMENT; ++t) sum += l[t * ld + n];
 #pragma unroll
-        for (int t = 0; t < SEGMENT; ++t) {
-            const int at = (t0 + t) * ld + n;
-            sum += l[at];
-            scaled[at] = x[at] * expf(sum);
+            for (int t = 0; t < SEGMENT; ++t) {
+                const int at = (segment * SEGMENT + t) * ld + n;
+                sum += l[at];
+                scaled[at] = x[at] * exp2f(sum);
+            }
         }
-    }
 }
 
 // ---- first kernel, plain ------------------------------------------------------------------------------------------
@@ -270,8 +311,8 @@ channel_keys_kernel(const float* __restrict__ rows, const float* __restrict__ lo
 
 // ---- first kernel, delta rule ----------------------------------------------------------------------------------------
 // Also w_rows[t][h * dim + n] = W and u[t][h * vdim + e] = U0.  A block per (chunk, head, sequence).
-template <int CH>
-__global__ void __launch_bounds__(CS_OUT_THREADS)
+template <int CH, int BLOCKS>
+__global__ void __launch_bounds__(CS_PREPARE_THREADS, BLOCKS)
 delta_prepare_kernel(const float* __restrict__ rows, const float* __restrict__ log_decay, const float* __restrict__ beta_rows,
                      int beta_stride, float* __restrict__ keys, float* __restrict__ factors, float* __restrict__ w_rows,
                      float* __restrict__ u, int max_chunks, const ChannelShape shape, const int* __restrict__ cu_q) {
@@ -284,35 +325,37 @@ delta_prepare_kernel(const float* __restrict__ rows, const float* __restrict__ l
     float* l = k + CH * ld;                // [CH][ld]
     float* scaled = l + CH * ld;           // [CH][ld]
     float* A = scaled + CH * ld;           // [CH][LDW]
-    float* beta = A + CH * LDW;            // [CH]
+    float* AT = A + CH * LDW;              // [CH][LDW]: transposed, times beta of the row
+    float* beta = AT + CH * LDW;           // [CH]
     const int chunk = blockIdx.x, head = blockIdx.y, s = blockIdx.z, g = head / (H / shape.groups);
     const int first = cu_q[s] + chunk * CH, L = min(CH, cu_q[s + 1] - first);
     if (L <= 0) return;
     const int channels = H * N;
-    load_chunk<CH, CS_OUT_THREADS>(k, ld, rows + (size_t)first * shape.row_stride + shape.k_at + g * N, shape.row_stride, L, N, n_pad);
-    load_chunk<CH, CS_OUT_THREADS>(l, ld, log_decay + (size_t)first * channels + head * N, channels, L, N, n_pad);
+    const RowPlace one = row_place<CS_PREPARE_THREADS>(n_pad), four = row_place<CS_PREPARE_THREADS>(n_pad >> 2);
+    load_chunk<CH>(k, ld, rows + (size_t)first * shape.row_stride + shape.k_at + g * N, shape.row_stride, L, N, n_pad, one, four);
+    load_chunk<CH>(l, ld, log_decay + (size_t)first * channels + head * N, channels, L, N, n_pad, one, four, CS_LOG2E);
     if (threadIdx.x < CH) beta[threadIdx.x] = threadIdx.x < L ? cs_sigmoid(beta_rows[(size_t)(first + threadIdx.x) * beta_stride + head]) : 0.0f;
     __syncthreads();
-    unit_rows<CH, CS_OUT_THREADS>(k, ld, n_pad, shape.unit_eps, 1.0f);
+    unit_rows<CH, CS_PREPARE_THREADS>(k, ld, n_pad, shape.unit_eps, 1.0f);
     __syncthreads();
     // the decayed keys and the chunk's factor
-    for (int n = threadIdx.x; n < N; n += CS_OUT_THREADS) {
+    for (int n = threadIdx.x; n < N; n += CS_PREPARE_THREADS) {
         float sum = 0.0f;
         for (int t = CH - 1; t >= 0; --t) {
-            if (t < L) keys[(size_t)(first + t) * channels + head * N + n] = k[t * ld + n] * expf(sum);
+            if (t < L) keys[(size_t)(first + t) * channels + head * N + n] = k[t * ld + n] * exp2f(sum);
             sum += l[t * ld + n];
         }
-        factors[((size_t)s * max_chunks + chunk) * channels + head * N + n] = expf(sum);
+        factors[((size_t)s * max_chunks + chunk) * channels + head * N + n] = exp2f(sum);
     }
-    decayed_products<CH, CS_OUT_THREADS>(A, scaled, k, k, l, ld, n_pad);
-    scale_from_start<CH, CS_OUT_THREADS>(scaled, k, l, ld, n_pad);
-    for (int idx = threadIdx.x; idx < CH * CH; idx += CS_OUT_THREADS) {
-        const int i = idx / CH, j = idx - i * CH;
-        A[i * LDW + j] = j < i ? A[i * LDW + j] * beta[i] : 0.0f;
+    decayed_products<CH, CS_PREPARE_THREADS>(A, scaled, k, k, l, ld, n_pad, one);
+    scale_from_start<CH>(scaled, k, l, ld, n_pad, one);
+    for (int idx = threadIdx.x; idx < CH * CH; idx += CS_PREPARE_THREADS) {
+        const int j = idx / CH, i = idx - j * CH;
+        AT[j * LDW + i] = j < i ? A[i * LDW + j] * beta[i] : 0.0f;
     }
     __syncthreads();
-    // (I + A) X = beta [K * E | V]: a thread takes a column from the top down
-    for (int column = threadIdx.x; column < N + P; column += CS_OUT_THREADS) {
+    // (I + A) X = beta [K * E | V]: a thread takes a column, and a row that is done is taken off all rows below it
+    for (int column = threadIdx.x; column < N + P; column += CS_PREPARE_THREADS) {
         const bool is_key = column < N;
         const int c = is_key ? column : column - N;
         const float* v = rows + (size_t)first * shape.row_stride + shape.v_at + head * P + c;
@@ -320,17 +363,15 @@ delta_prepare_kernel(const float* __restrict__ rows, const float* __restrict__ l
 #pragma unroll
         for (int i = 0; i < CH; ++i) x[i] = i < L ? beta[i] * (is_key ? scaled[i * ld + c] : v[(size_t)i * shape.row_stride]) : 0.0f;
 #pragma unroll
-        for (int i = 1; i < CH; ++i) {
-            float r = x[i];
+        for (int j = 0; j < CH - 1; ++j) {
 #pragma unroll
-            for (int j = 0; j < i; j += 4) {
-                const float4 a = *(const float4*)(A + i * LDW + j);        // (zero from the diagonal on)
-                r = fmaf(-a.x, x[j], r);
-                if (j + 1 < i) r = fmaf(-a.y, x[j + 1], r);
-                if (j + 2 < i) r = fmaf(-a.z, x[j + 2], r);
-                if (j + 3 < i) r = fmaf(-a.w, x[j + 3], r);
+            for (int i = (j + 1) & ~3; i < CH; i += 4) {
+                const float4 a = *(const float4*)(AT + j * LDW + i);       // (zero up to the diagonal)
+                if (i > j) x[i] = fmaf(-a.x, x[j], x[i]);
+                if (i + 1 > j) x[i + 1] = fmaf(-a.y, x[j], x[i + 1]);
+                if (i + 2 > j) x[i + 2] = fmaf(-a.z, x[j], x[i + 2]);
+                if (i + 3 > j) x[i + 3] = fmaf(-a.w, x[j], x[i + 3]);
             }
-            x[i] = r;
         }
         float* to = is_key ? w_rows + (size_t)first * channels + head * N + c : u + (size_t)first * H * P + (size_t)head * P + c;
         const size_t stride = is_key ? channels : H * P;
@@ -341,9 +382,10 @@ delta_prepare_kernel(const float* __restrict__ rows, const float* __restrict__ l
 }
 
 // ---- second kernel: the walk over a sequence's chunks ---------------------------------------------------------------
-// A block per (slice of C value columns, head, sequence); a thread owns four key channels by two columns of S per 64
+// A block per (slice of C value columns, head, sequence); a thread owns two key channels by two columns of S per 64
 // channels.  states [seqs][max_chunks][heads][dim][vdim] gets the state before every chunk; with the delta rule
-// u [tokens][heads * vdim] turns from U0 into U.  The next chunk's rows are on their way while one is worked on.
+// u [tokens][heads * vdim] turns from U0 into U.  The next chunks' rows are on their way while one is worked on (a ring of two
+// or four).
 __device__ __forceinline__ void cs_copy16(float* dst, const float* src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
 }
@@ -351,31 +393,34 @@ __device__ __forceinline__ void cs_copy4(float* dst, const float* src) {
     asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
 }
 
-template <int THREADS>
-__device__ __forceinline__ void stage_rows(float* to, int ld, const float* from, size_t stride, int rows_there, int rows, int N, bool vec) {
-    if (vec) {
-        const int quads = N >> 2;
-        for (int idx = threadIdx.x; idx < rows * quads; idx += THREADS) {
-            const int t = idx / quads, n = (idx - t * quads) * 4;
-            if (t < rows_there) cs_copy16(to + t * ld + n, from + t * stride + n);
-            else *(float4*)(to + t * ld + n) = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-        }
-    } else {
-        for (int idx = threadIdx.x; idx < rows * N; idx += THREADS) {
-            const int t = idx / N, n = idx - t * N;
-            if (t < rows_there) cs_copy4(to + t * ld + n, from + t * stride + n);
-            else to[t * ld + n] = 0.0f;
+// `rows` rows of `items` 16-byte (vec) or 4-byte pieces, those past `there` zero; `place` over a row's pieces.
+__device__ __forceinline__ void stage_rows(float* to, int ld, const float* from, size_t stride, int there, int rows, int items, bool vec,
+                                           const RowPlace& place) {
+    const int each = vec ? 4 : 1;
+    for (int item = place.item; item < items; item += place.lanes) {
+        float* at = to + place.row * ld + item * each;
+        const float* src = from + place.row * stride + item * each;
+        for (int t = place.row; t < rows; t += place.rows) {
+            if (vec) {
+                if (t < there) cs_copy16(at, src);
+                else *(float4*)at = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            } else {
+                if (t < there) cs_copy4(at, src);
+                else *at = 0.0f;
+            }
+            at += place.rows * ld;
+            src += place.rows * stride;
         }
     }
 }
 
 template <int CH, int C, bool DELTA>
-__global__ void __launch_bounds__(C * 8)
+__global__ void __launch_bounds__(C * 16)
 channel_walk_kernel(const float* __restrict__ keys, const float* __restrict__ factors, const float* __restrict__ w_rows, float* u,
-                    const float* __restrict__ values, int value_stride, float* __restrict__ states, int max_chunks,
+                    const float* __restrict__ values, int value_stride, float* __restrict__ states, int max_chunks, int stages,
                     const ChannelShape shape, const ChannelBatch batch) {
     extern __shared__ __align__(16) float cs_smem[];
-    constexpr int THREADS = C * 8, TOK = CH / 16;
+    constexpr int THREADS = C * 16;
     pdl_launch_dependents();
     pdl_wait();
     const int H = shape.heads, N = shape.dim, P = shape.vdim, n_pad = cs_pad(N), ld = n_pad + 4, channels = H * N;
@@ -393,71 +438,73 @@ channel_walk_kernel(const float* __restrict__ keys, const float* __restrict__ fa
         const int n = idx / C, c = idx - n * C;
         S[idx] = p_first > 0 && n < N && c < width ? before[(size_t)n * P + c] : 0.0f;
     }
-    for (int idx = threadIdx.x; idx < 2 * set; idx += THREADS) sets[idx] = 0.0f;        // (what pads stays zero)
+    for (int idx = threadIdx.x; idx < stages * set; idx += THREADS) sets[idx] = 0.0f;        // (what pads stays zero)
     __syncthreads();
     const bool vec_n = (N & 3) == 0;
     const int u_stride = DELTA ? H * P : value_stride;
     const float* u_from = DELTA ? u + (size_t)head * P + e0 : values + (size_t)head * P + e0;
     const bool vec_u = ((u_stride | P | e0) & 3) == 0 && ((uintptr_t)u_from & 15) == 0 && (width & 3) == 0;
+    const int n_items = vec_n ? N >> 2 : N, u_items = vec_u ? width >> 2 : width;
+    const RowPlace n_place = row_place<THREADS>(n_items), u_place = row_place<THREADS>(u_items);
     auto stage = [&](int which, int chunk) {
         float* kh = sets + which * set;
         const int t0 = first + chunk * CH, L = min(CH, count - chunk * CH);
-        stage_rows<THREADS>(kh, ld, keys + (size_t)t0 * channels + head * N, channels, L, CH, N, vec_n);
-        if (DELTA) stage_rows<THREADS>(kh + CH * ld, ld, w_rows + (size_t)t0 * channels + head * N, channels, L, CH, N, vec_n);
+        stage_rows(kh, ld, keys + (size_t)t0 * channels + head * N, channels, L, CH, n_items, vec_n, n_place);
+        if (DELTA) stage_rows(kh + CH * ld, ld, w_rows + (size_t)t0 * channels + head * N, channels, L, CH, n_items, vec_n, n_place);
         float* ut = kh + CH * ld * (DELTA ? 2 : 1);
-        stage_rows<THREADS>(ut, C, u_from + (size_t)t0 * u_stride, u_stride, L, CH, width, vec_u);
-        stage_rows<THREADS>(ut + CH * C, n_pad, factors + ((size_t)s * max_chunks + chunk) * channels + head * N, 0, 1, 1, N, vec_n);
-        asm volatile("cp.async.commit_group;" ::: "memory");
+        stage_rows(ut, C, u_from + (size_t)t0 * u_stride, u_stride, L, CH, u_items, vec_u, u_place);
+        stage_rows(ut + CH * C, n_pad, factors + ((size_t)s * max_chunks + chunk) * channels + head * N, 0, 1, 1, n_items, vec_n, n_place);
     };
     const int rg = threadIdx.x / (C / 2), c0 = (threadIdx.x % (C / 2)) * 2;
     const int chunks = (count + CH - 1) / CH;
     const bool pairs = (P & 1) == 0;
-    stage(0, 0);
+    for (int ahead = 0; ahead < stages - 1; ++ahead) {
+        if (ahead < chunks) stage(ahead, ahead);
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    }
     for (int chunk = 0; chunk < chunks; ++chunk) {
-        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        if (stages == 4) asm volatile("cp.async.wait_group 2;" ::: "memory");
+        else asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();                   // this chunk's rows are there, and everybody is done with the one before
-        if (chunk + 1 < chunks) stage((chunk + 1) & 1, chunk + 1);
-        float* kh = sets + (chunk & 1) * set;
+        if (chunk + stages - 1 < chunks) stage((chunk + stages - 1) & (stages - 1), chunk + stages - 1);
+        asm volatile("cp.async.commit_group;" ::: "memory");
+        float* kh = sets + (chunk & (stages - 1)) * set;
         float* w = kh + CH * ld;
         float* ut = kh + CH * ld * (DELTA ? 2 : 1);
         const float* f = ut + CH * C;
         const int t0 = first + chunk * CH, L = min(CH, count - chunk * CH);
         if (DELTA) {
-            float acc[TOK][2];
-#pragma unroll
-            for (int a = 0; a < TOK; ++a) { acc[a][0] = ut[(rg * TOK + a) * C + c0]; acc[a][1] = ut[(rg * TOK + a) * C + c0 + 1]; }
+            if (rg < CH) {                 // a token by two columns a thread
+                float2 acc = *(const float2*)(ut + rg * C + c0);
+                const float* w_row = w + rg * ld;
 #pragma unroll 4
-            for (int n = 0; n < n_pad; n += 4) {
-                float2 sv[4];
-#pragma unroll
-                for (int x = 0; x < 4; ++x) sv[x] = *(const float2*)(S + (n + x) * C + c0);
-#pragma unroll
-                for (int a = 0; a < TOK; ++a) {
-                    const float4 wv = *(const float4*)(w + (rg * TOK + a) * ld + n);
-                    acc[a][0] = fmaf(-wv.x, sv[0].x, acc[a][0]); acc[a][1] = fmaf(-wv.x, sv[0].y, acc[a][1]);
-                    acc[a][0] = fmaf(-wv.y, sv[1].x, acc[a][0]); acc[a][1] = fmaf(-wv.y, sv[1].y, acc[a][1]);
-                    acc[a][0] = fmaf(-wv.z, sv[2].x, acc[a][0]); acc[a][1] = fmaf(-wv.z, sv[2].y, acc[a][1]);
-                    acc[a][0] = fmaf(-wv.w, sv[3].x, acc[a][0]); acc[a][1] = fmaf(-wv.w, sv[3].y, acc[a][1]);
+                for (int n = 0; n < n_pad; n += 4) {
+                    const float4 wv = *(const float4*)(w_row + n);
+                    const float2 s0 = *(const float2*)(S + n * C + c0), s1 = *(const float2*)(S + (n + 1) * C + c0);
+                    const float2 s2 = *(const float2*)(S + (n + 2) * C + c0), s3 = *(const float2*)(S + (n + 3) * C + c0);
+                    acc.x = fmaf(-wv.x, s0.x, acc.x); acc.y = fmaf(-wv.x, s0.y, acc.y);
+                    acc.x = fmaf(-wv.y, s1.x, acc.x); acc.y = fmaf(-wv.y, s1.y, acc.y);
+                    acc.x = fmaf(-wv.z, s2.x, acc.x); acc.y = fmaf(-wv.z, s2.y, acc.y);
+                    acc.x = fmaf(-wv.w, s3.x, acc.x); acc.y = fmaf(-wv.w, s3.y, acc.y);
                 }
-            }
-#pragma unroll
-            for (int a = 0; a < TOK; ++a) {
-                const int t = rg * TOK + a;
-                *(float2*)(ut + t * C + c0) = make_float2(acc[a][0], acc[a][1]);       // (nobody else reads or writes these yet)
-                if (t >= L) continue;
-                float* to = u + (size_t)(t0 + t) * H * P + (size_t)head * P + e0 + c0;
-                if (c0 < width) to[0] = acc[a][0];
-                if (c0 + 1 < width) to[1] = acc[a][1];
+                *(float2*)(ut + rg * C + c0) = acc;                        // (nobody else reads or writes these yet)
+                if (rg < L) {
+                    float* to = u + (size_t)(t0 + rg) * H * P + (size_t)head * P + e0 + c0;
+                    if (pairs && c0 + 1 < width) *(float2*)to = acc;
+                    else {
+                        if (c0 < width) to[0] = acc.x;
+                        if (c0 + 1 < width) to[1] = acc.y;
+                    }
+                }
             }
             __syncthreads();               // U is there, and everybody is done with S as it was
         }
         float* kept = states + (((size_t)s * max_chunks + chunk) * H + head) * (size_t)N * P + e0 + c0;
-        for (int n0 = rg * 4; n0 < n_pad; n0 += 64) {
-            float2 sv[4];
-            const float4 fv = *(const float4*)(f + n0);
-            const float fs[4] = {fv.x, fv.y, fv.z, fv.w};
+        for (int n0 = rg * 2; n0 < n_pad; n0 += 64) {
+            float2 sv[2];
+            const float2 fv = *(const float2*)(f + n0);
 #pragma unroll
-            for (int x = 0; x < 4; ++x) {
+            for (int x = 0; x < 2; ++x) {
                 sv[x] = *(const float2*)(S + (n0 + x) * C + c0);
                 if (n0 + x < N) {
                     if (pairs && c0 + 1 < width) *(float2*)(kept + (size_t)(n0 + x) * P) = sv[x];
@@ -466,27 +513,25 @@ channel_walk_kernel(const float* __restrict__ keys, const float* __restrict__ fa
                         if (c0 + 1 < width) kept[(size_t)(n0 + x) * P + 1] = sv[x].y;
                     }
                 }
-                sv[x].x *= fs[x];
-                sv[x].y *= fs[x];
+                sv[x].x *= x == 0 ? fv.x : fv.y;
+                sv[x].y *= x == 0 ? fv.x : fv.y;
             }
-#pragma unroll 8
+#pragma unroll
             for (int j = 0; j < CH; ++j) {
-                const float4 kv = *(const float4*)(kh + j * ld + n0);
+                const float2 kv = *(const float2*)(kh + j * ld + n0);
                 const float2 uv = *(const float2*)(ut + j * C + c0);
                 sv[0].x = fmaf(kv.x, uv.x, sv[0].x); sv[0].y = fmaf(kv.x, uv.y, sv[0].y);
                 sv[1].x = fmaf(kv.y, uv.x, sv[1].x); sv[1].y = fmaf(kv.y, uv.y, sv[1].y);
-                sv[2].x = fmaf(kv.z, uv.x, sv[2].x); sv[2].y = fmaf(kv.z, uv.y, sv[2].y);
-                sv[3].x = fmaf(kv.w, uv.x, sv[3].x); sv[3].y = fmaf(kv.w, uv.y, sv[3].y);
             }
 #pragma unroll
-            for (int x = 0; x < 4; ++x) *(float2*)(S + (n0 + x) * C + c0) = sv[x];
+            for (int x = 0; x < 2; ++x) *(float2*)(S + (n0 + x) * C + c0) = sv[x];
         }
     }
     // (a thread writes what it owns)
     float* after = slot + (size_t)(p_last & 1) * half + mine + c0;
-    for (int n0 = rg * 4; n0 < N; n0 += 64)
+    for (int n0 = rg * 2; n0 < N; n0 += 64)
 #pragma unroll
-        for (int x = 0; x < 4; ++x) {
+        for (int x = 0; x < 2; ++x) {
             if (n0 + x >= N) continue;
             const float2 sv = *(const float2*)(S + (n0 + x) * C + c0);
             if (c0 < width) after[(size_t)(n0 + x) * P] = sv.x;
@@ -495,15 +540,15 @@ channel_walk_kernel(const float* __restrict__ keys, const float* __restrict__ fa
 }
 
 // ---- third kernel: outputs ---------------------------------------------------------------------------------------------
-// A block per (chunk, head, sequence): threads in 8 x 16, each with CH / 8 tokens and four columns of a tile of 64.
+// A block per (chunk, head, sequence): threads in 16 x 16, each with CH / 16 tokens and four columns of a tile of 64.
 // values: the row of (token, head) at values + token * value_stride + head * vdim (v, or the delta rule's U).
 template <int CH>
-__global__ void __launch_bounds__(CS_OUT_THREADS)
+__global__ void __launch_bounds__(CS_OUT_THREADS, 4)
 channel_output_kernel(const float* __restrict__ rows, const float* __restrict__ log_decay, const float* __restrict__ values,
                       int value_stride, const float* __restrict__ states, float* __restrict__ out, int max_chunks,
                       const ChannelShape shape, const int* __restrict__ cu_q) {
     extern __shared__ __align__(16) float cs_smem[];
-    constexpr int LDW = CH + 4, RI = CH / 8;
+    constexpr int LDW = CH + 4, RI = CH / 16;
     pdl_launch_dependents();
     pdl_wait();
     const int H = shape.heads, N = shape.dim, P = shape.vdim, n_pad = cs_pad(N), ld = n_pad + 4;
@@ -518,9 +563,10 @@ channel_output_kernel(const float* __restrict__ rows, const float* __restrict__ 
     const int first = cu_q[s] + chunk * CH, L = min(CH, cu_q[s + 1] - first);
     if (L <= 0) return;
     const float* base = rows + (size_t)first * shape.row_stride;
-    load_chunk<CH, CS_OUT_THREADS>(q, ld, base + shape.q_at + g * N, shape.row_stride, L, N, n_pad);
-    load_chunk<CH, CS_OUT_THREADS>(k, ld, base + shape.k_at + g * N, shape.row_stride, L, N, n_pad);
-    load_chunk<CH, CS_OUT_THREADS>(l, ld, log_decay + (size_t)first * H * N + head * N, (size_t)H * N, L, N, n_pad);
+    const RowPlace one = row_place<CS_OUT_THREADS>(n_pad), four = row_place<CS_OUT_THREADS>(n_pad >> 2);
+    load_chunk<CH>(q, ld, base + shape.q_at + g * N, shape.row_stride, L, N, n_pad, one, four);
+    load_chunk<CH>(k, ld, base + shape.k_at + g * N, shape.row_stride, L, N, n_pad, one, four);
+    load_chunk<CH>(l, ld, log_decay + (size_t)first * H * N + head * N, (size_t)H * N, L, N, n_pad, one, four, CS_LOG2E);
     for (int idx = threadIdx.x; idx < CH * LDW; idx += CS_OUT_THREADS) w[idx] = 0.0f;
     __syncthreads();
     unit_rows<CH, CS_OUT_THREADS>(q, ld, n_pad, shape.unit_eps, shape.q_scale);
@@ -535,8 +581,8 @@ channel_output_kernel(const float* __restrict__ rows, const float* __restrict__ 
         for (int offset = PARTS >> 1; offset > 0; offset >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, offset);
         if (part == 0) w[i * LDW + i] = acc;
     }
-    decayed_products<CH, CS_OUT_THREADS>(w, scaled, q, k, l, ld, n_pad);
-    scale_from_start<CH, CS_OUT_THREADS>(scaled, q, l, ld, n_pad);
+    decayed_products<CH, CS_OUT_THREADS>(w, scaled, q, k, l, ld, n_pad, one);
+    scale_from_start<CH>(scaled, q, l, ld, n_pad, one);
     const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4, i0 = ty * RI;
     const float* before = states + (((size_t)s * max_chunks + chunk) * H + head) * (size_t)N * P;
     const float* vbase = values + (size_t)first * value_stride + (size_t)head * P;
@@ -902,17 +948,17 @@ static size_t cs_output_smem(int ch, int dim) {
 }
 
 static size_t cs_prepare_smem(int ch, int dim) {
-    return (size_t)(3 * ch * (((dim + 3) & ~3) + 4) + ch * (ch + 4) + ch) * sizeof(float);
+    return (size_t)(3 * ch * (((dim + 3) & ~3) + 4) + 2 * ch * (ch + 4) + ch) * sizeof(float);
 }
 
-static size_t cs_walk_smem(int ch, int cols, int dim, bool delta) {
+static size_t cs_walk_smem(int ch, int cols, int dim, bool delta, int stages) {
     const int n_pad = (dim + 3) & ~3, ld = n_pad + 4;
-    return (size_t)(n_pad * cols + 2 * (ch * ld * (delta ? 2 : 1) + ch * cols + n_pad)) * sizeof(float);
+    return (size_t)(n_pad * cols + stages * (ch * ld * (delta ? 2 : 1) + ch * cols + n_pad)) * sizeof(float);
 }
 
 // The longest chunk whose tiles fit: 32 tokens or 16.
 static int cs_chunk(int dim) {
-    return cs_output_smem(32, dim) <= 200 * 1024 && cs_walk_smem(32, 16, dim, true) <= 200 * 1024 ? 32 : 16;
+    return cs_output_smem(32, dim) <= 200 * 1024 && cs_walk_smem(32, 16, dim, true, 2) <= 200 * 1024 ? 32 : 16;
 }
 
 static int cs_check(const char* name, const ChannelShape& shape, const ChannelBatch& batch, long long state_floats) {
@@ -947,8 +993,9 @@ SKV_EXPORT int skv_low_rank(const float* x, int x_stride, int rank, const void* 
     const int tok = many ? 16 : 4;
     const size_t smem = (size_t)rank * tok * sizeof(float);
     if (smem > 48 * 1024) return fail(name, "the rank is too large");
-    auto kernel = many ? low_rank_kernel<skv_t, 16> : low_rank_kernel<skv_t, 4>;
-    return launch_pdl(name, kernel, dim3((n + tok - 1) / tok, (channels + 255) / 256), dim3(256), smem, stream, x, x_stride,
+    const int each = many && channels % 2 == 0 && (((uintptr_t)wt | (uintptr_t)out) & 7) == 0 ? 2 : 1;
+    auto kernel = each == 2 ? low_rank_kernel<skv_t, 16, 2> : (many ? low_rank_kernel<skv_t, 16, 1> : low_rank_kernel<skv_t, 4, 1>);
+    return launch_pdl(name, kernel, dim3((n + tok - 1) / tok, (channels + 256 * each - 1) / (256 * each)), dim3(256), smem, stream, x, x_stride,
                       rank, (const skv_t*)wt, end, out, n, channels);
 }
 
@@ -990,9 +1037,11 @@ SKV_EXPORT int skv_channel_state(const float* rows, int row_stride, int q_at, in
     const dim3 grid(max_chunks, heads, n_seqs);
     if (delta) {
         const size_t smem = cs_prepare_smem(ch, dim);
-        auto kernel = ch == 32 ? delta_prepare_kernel<32> : delta_prepare_kernel<16>;
+        // (one turn of columns: more blocks an SM, with fewer registers; several: fewer)
+        auto kernel = ch == 32 ? (dim + vdim <= CS_PREPARE_THREADS ? delta_prepare_kernel<32, 5> : delta_prepare_kernel<32, 3>)
+                               : delta_prepare_kernel<16, 3>;
         if (int code = cs_reserve((const void*)kernel, smem, name)) return code;
-        if (int code = launch_pdl(name, kernel, grid, dim3(CS_OUT_THREADS), smem, stream, rows, log_decay, beta_rows, beta_stride,
+        if (int code = launch_pdl(name, kernel, grid, dim3(CS_PREPARE_THREADS), smem, stream, rows, log_decay, beta_rows, beta_stride,
                                   keys, factors, w_rows, u, max_chunks, shape, cu_q))
             return code;
     } else {
@@ -1005,17 +1054,21 @@ SKV_EXPORT int skv_channel_state(const float* rows, int row_stride, int q_at, in
     const int value_stride = delta ? heads * vdim : row_stride;
     {
         // slices of 32 value columns where that gives blocks enough, else 16
-        const bool wide = (long long)((vdim + 31) / 32) * heads * n_seqs >= 2 * sm_count() && cs_walk_smem(ch, 32, dim, delta) <= 200 * 1024;
+        const bool wide = 4LL * ((vdim + 31) / 32) * heads * n_seqs >= 3 * sm_count() && cs_walk_smem(ch, 32, dim, delta, 2) <= 200 * 1024;
         const int cols = wide ? 32 : 16;
-        const size_t smem = cs_walk_smem(ch, cols, dim, delta);
+        // a ring of four where no block has to wait for another's shared memory
+        const size_t four = cs_walk_smem(ch, cols, dim, delta, 4);
+        const bool alone = (long long)((vdim + cols - 1) / cols) * heads * n_seqs <= sm_count();
+        const int stages = max_chunks > 2 && four <= (alone ? 200 : 100) * 1024 ? 4 : 2;
+        const size_t smem = cs_walk_smem(ch, cols, dim, delta, stages);
         auto kernel = ch == 32 ? (wide ? (delta ? channel_walk_kernel<32, 32, true> : channel_walk_kernel<32, 32, false>)
                                        : (delta ? channel_walk_kernel<32, 16, true> : channel_walk_kernel<32, 16, false>))
                                : (wide ? (delta ? channel_walk_kernel<16, 32, true> : channel_walk_kernel<16, 32, false>)
                                        : (delta ? channel_walk_kernel<16, 16, true> : channel_walk_kernel<16, 16, false>));
         if (int code = cs_reserve((const void*)kernel, smem, name)) return code;
-        if (int code = launch_pdl(name, kernel, dim3((vdim + cols - 1) / cols, heads, n_seqs), dim3(cols * 8), smem, stream,
+        if (int code = launch_pdl(name, kernel, dim3((vdim + cols - 1) / cols, heads, n_seqs), dim3(cols * 16), smem, stream,
                                   (const float*)keys, (const float*)factors, (const float*)w_rows, u, values, value_stride, states,
-                                  max_chunks, shape, batch))
+                                  max_chunks, stages, shape, batch))
             return code;
     }
     const size_t smem = cs_output_smem(ch, dim);

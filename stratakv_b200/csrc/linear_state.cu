@@ -767,7 +767,7 @@ step_sizes_kernel(const float* __restrict__ rows, int row_stride, int dt_at, con
 // [tokens][heads]: what linear_state reads.  The state of a slot holds m twice, [2][heads] from m_offset on, by the parity of
 // the last position.  A block per (head, sequence); a thread takes EG_EACH neighbouring tokens.  A run of tokens turns m into
 // max(F + m, M) with F the sum of its f, and two runs behind one another make another such pair, which the block scans.
-constexpr int EG_EACH = 4;
+constexpr int EG_EACH = 8;
 
 struct GateRun { float F, M; };
 __device__ __forceinline__ GateRun behind_run(GateRun a, GateRun b) { return {a.F + b.F, fmaxf(b.F + a.M, b.M)}; }

@@ -90,10 +90,14 @@ __global__ void rmsnorm_add_rows_kernel(const float* __restrict__ y, const float
         const int i = threadIdx.x + u * blockDim.x;
         if (i < quads) {
             const float4 g = next_gamma ? ((const float4*)next_gamma)[i] : make_float4(1.0f, 1.0f, 1.0f, 1.0f);
-            out_row[4 * i] = from_float<T>(stream[u].x * next_inverse * g.x);
-            out_row[4 * i + 1] = from_float<T>(stream[u].y * next_inverse * g.y);
-            out_row[4 * i + 2] = from_float<T>(stream[u].z * next_inverse * g.z);
-            out_row[4 * i + 3] = from_float<T>(stream[u].w * next_inverse * g.w);
+            const float4 v = make_float4(stream[u].x * next_inverse * g.x, stream[u].y * next_inverse * g.y,
+                                         stream[u].z * next_inverse * g.z, stream[u].w * next_inverse * g.w);
+            if (sizeof(T) == 4) {
+                *(float4*)(out_row + 4 * i) = v;
+            } else {
+                const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+                *(uint2*)(out_row + 4 * i) = make_uint2(*(const uint32_t*)&lo, *(const uint32_t*)&hi);
+            }
         }
     }
 }
@@ -295,7 +299,7 @@ SKV_EXPORT int skv_rmsnorm_add(const float* y, const float* gamma, float eps, fl
     if (next_gamma && !next_out) return fail("skv_rmsnorm_add", "the next norm needs a place for its result");
     const int threads = stream_threads(hidden);
     const bool aligned = hidden % 4 == 0 &&
-                         (((uintptr_t)y | (uintptr_t)x | (uintptr_t)gamma | (uintptr_t)next_gamma) & 15) == 0;
+                         (((uintptr_t)y | (uintptr_t)x | (uintptr_t)gamma | (uintptr_t)next_gamma | (uintptr_t)next_out) & 15) == 0;
     if (aligned && hidden <= 4 * 4 * threads)
         return launch_pdl("skv_rmsnorm_add", rmsnorm_add_rows_kernel<skv_t, 4>, dim3(n_rows), dim3(threads), 0, stream, y,
                           gamma, eps, x, next_gamma, next_eps, (skv_t*)next_out, hidden);
