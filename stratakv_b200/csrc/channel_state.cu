@@ -393,14 +393,31 @@ __device__ __forceinline__ void cs_copy4(float* dst, const float* src) {
     asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
 }
 
-// `rows` rows of `items` 16-byte (vec) or 4-byte pieces, those past `there` zero; `place` over a row's pieces.
-__device__ __forceinline__ void stage_rows(float* to, int ld, const float* from, size_t stride, int there, int rows, int items, bool vec,
-                                           const RowPlace& place) {
-    const int each = vec ? 4 : 1;
-    for (int item = place.item; item < items; item += place.lanes) {
-        float* at = to + place.row * ld + item * each;
-        const float* src = from + place.row * stride + item * each;
-        for (int t = place.row; t < rows; t += place.rows) {
+// What a thread copies of an array's rows for every chunk: made once, so that a chunk costs it little but the copies.  Rows of
+// `items` pieces of 16 bytes (vec) or of 4.
+struct StagePlan {
+    const float* src;                      // this thread's piece of its first row of chunk 0
+    int dst;                               // where it goes within the array's place of a stage
+    int row, rows;                         // its first row and the rows between its turns
+    size_t src_step;
+    int dst_step;
+    int item, items, lanes;                // its first piece of a row, the pieces, and those between its turns within a row
+};
+
+template <int THREADS>
+__device__ __forceinline__ StagePlan stage_plan(const float* from, size_t stride, int ld, int items, bool vec) {
+    const RowPlace place = row_place<THREADS>(items);
+    const int each = vec ? 4 : 1, row = min(place.row, 1 << 14);
+    return {from + (size_t)row * stride + place.item * each, row * ld + place.item * each, row, place.rows, place.rows * stride, place.rows * ld,
+            place.item, items, place.lanes};
+}
+
+// Rows [0, rows) of a chunk that starts `skip` floats into the array; those past `there` become zero.
+__device__ __forceinline__ void stage_rows(float* to, const StagePlan& plan, size_t skip, int there, int rows, bool vec) {
+    for (int more = 0; plan.item + more < plan.items; more += plan.lanes) {        // (once, unless a row has more pieces than threads)
+        float* at = to + plan.dst + more * (vec ? 4 : 1);
+        const float* src = plan.src + skip + more * (vec ? 4 : 1);
+        for (int t = plan.row; t < rows; t += plan.rows) {
             if (vec) {
                 if (t < there) cs_copy16(at, src);
                 else *(float4*)at = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
@@ -408,8 +425,8 @@ __device__ __forceinline__ void stage_rows(float* to, int ld, const float* from,
                 if (t < there) cs_copy4(at, src);
                 else *at = 0.0f;
             }
-            at += place.rows * ld;
-            src += place.rows * stride;
+            at += plan.dst_step;
+            src += plan.src_step;
         }
     }
 }
@@ -445,15 +462,23 @@ channel_walk_kernel(const float* __restrict__ keys, const float* __restrict__ fa
     const float* u_from = DELTA ? u + (size_t)head * P + e0 : values + (size_t)head * P + e0;
     const bool vec_u = ((u_stride | P | e0) & 3) == 0 && ((uintptr_t)u_from & 15) == 0 && (width & 3) == 0;
     const int n_items = vec_n ? N >> 2 : N, u_items = vec_u ? width >> 2 : width;
-    const RowPlace n_place = row_place<THREADS>(n_items), u_place = row_place<THREADS>(u_items);
+    const size_t chunk_keys = (size_t)CH * channels, chunk_values = (size_t)CH * u_stride;
+    const StagePlan key_plan = stage_plan<THREADS>(keys + (size_t)first * channels + head * N, channels, ld, n_items, vec_n);
+    const StagePlan value_plan = stage_plan<THREADS>(u_from + (size_t)first * u_stride, u_stride, C, u_items, vec_u);
+    const StagePlan factor_plan = stage_plan<THREADS>(factors + (size_t)s * max_chunks * channels + head * N, 0, n_pad, n_items, vec_n);
+    const float* w_first = DELTA ? w_rows + (key_plan.src - keys) : nullptr;
     auto stage = [&](int which, int chunk) {
         float* kh = sets + which * set;
-        const int t0 = first + chunk * CH, L = min(CH, count - chunk * CH);
-        stage_rows(kh, ld, keys + (size_t)t0 * channels + head * N, channels, L, CH, n_items, vec_n, n_place);
-        if (DELTA) stage_rows(kh + CH * ld, ld, w_rows + (size_t)t0 * channels + head * N, channels, L, CH, n_items, vec_n, n_place);
+        const int L = min(CH, count - chunk * CH);
+        stage_rows(kh, key_plan, chunk * chunk_keys, L, CH, vec_n);
+        if (DELTA) {
+            StagePlan w_plan = key_plan;
+            w_plan.src = w_first;
+            stage_rows(kh + CH * ld, w_plan, chunk * chunk_keys, L, CH, vec_n);
+        }
         float* ut = kh + CH * ld * (DELTA ? 2 : 1);
-        stage_rows(ut, C, u_from + (size_t)t0 * u_stride, u_stride, L, CH, u_items, vec_u, u_place);
-        stage_rows(ut + CH * C, n_pad, factors + ((size_t)s * max_chunks + chunk) * channels + head * N, 0, 1, 1, n_items, vec_n, n_place);
+        stage_rows(ut, value_plan, chunk * chunk_values, L, CH, vec_u);
+        stage_rows(ut + CH * C, factor_plan, (size_t)chunk * channels, 1, 1, vec_n);
     };
     const int rg = threadIdx.x / (C / 2), c0 = (threadIdx.x % (C / 2)) * 2;
     const int chunks = (count + CH - 1) / CH;
@@ -725,6 +750,19 @@ __host__ __device__ __forceinline__ int ms_smem_floats(int N, int P, int rank, i
     return 3 * ((N + 3) & ~3) + 3 * ((P + 3) & ~3) + ((rank + 3) & ~3) + (columns > wide ? columns : wide) + 40;
 }
 
+// Sums of three numbers over the block; every thread gets them.  `scratch` holds 24 floats and may be reused after a barrier.
+__device__ __forceinline__ float3 block_sum3(float a, float b, float c, float* scratch) {
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    a = warp_sum(a); b = warp_sum(b); c = warp_sum(c);
+    __syncthreads();
+    if (lane == 0) { scratch[3 * warp] = a; scratch[3 * warp + 1] = b; scratch[3 * warp + 2] = c; }
+    __syncthreads();
+    float3 sums = make_float3(0.0f, 0.0f, 0.0f);
+#pragma unroll
+    for (int w = 0; w < MS_THREADS / 32; ++w) { sums.x += scratch[3 * w]; sums.y += scratch[3 * w + 1]; sums.z += scratch[3 * w + 2]; }
+    return sums;
+}
+
 template <typename T, int VEC, int KIND>
 __global__ void __launch_bounds__(MS_THREADS)
 matrix_step_kernel(const float* __restrict__ rows, T* __restrict__ out, int out_stride, const MatrixStep a, const ChannelBatch batch) {
@@ -831,7 +869,8 @@ matrix_step_kernel(const float* __restrict__ rows, T* __restrict__ out, int out_
         for (int n = threadIdx.x; n < N; n += MS_THREADS) {
             sq = fmaf(q[n], q[n], sq); sk = fmaf(k[n], k[n], sk); qk = fmaf(q[n], k[n], qk);
         }
-        sq = block_sum(sq, scratch); sk = block_sum(sk, scratch); qk = block_sum(qk, scratch);
+        const float3 sums = block_sum3(sq, sk, qk, scratch);
+        sq = sums.x; sk = sums.y; qk = sums.z;
         const bool unit = a.shape.unit_eps >= 0.0f;
         const float fq = unit ? a.shape.q_scale / sqrtf(sq + a.shape.unit_eps) : a.shape.q_scale;
         const float fk = unit ? 1.0f / sqrtf(sk + a.shape.unit_eps) : 1.0f;

@@ -767,16 +767,16 @@ step_sizes_kernel(const float* __restrict__ rows, int row_stride, int dt_at, con
 // [tokens][heads]: what linear_state reads.  The state of a slot holds m twice, [2][heads] from m_offset on, by the parity of
 // the last position.  A block per (head, sequence); a thread takes EG_EACH neighbouring tokens.  A run of tokens turns m into
 // max(F + m, M) with F the sum of its f, and two runs behind one another make another such pair, which the block scans.
-constexpr int EG_EACH = 8;
+constexpr int EG_EACH = 4, EG_THREADS = 512;
 
 struct GateRun { float F, M; };
 __device__ __forceinline__ GateRun behind_run(GateRun a, GateRun b) { return {a.F + b.F, fmaxf(b.F + a.M, b.M)}; }
 
-__global__ void __launch_bounds__(LS_THREADS)
+__global__ void __launch_bounds__(EG_THREADS)
 exp_gates_kernel(const float* __restrict__ rows, int row_stride, int input_at, int forget_at, const float* __restrict__ input_bias,
                  const float* __restrict__ forget_bias, float cap, float* __restrict__ log_decay, float* __restrict__ key_scale,
                  float* __restrict__ floor, int heads, const LinearStateBatch batch) {
-    __shared__ GateRun warp_runs[LS_THREADS / 32];
+    __shared__ GateRun warp_runs[EG_THREADS / 32];
     __shared__ float carried;
     pdl_launch_dependents();
     pdl_wait();
@@ -787,7 +787,7 @@ exp_gates_kernel(const float* __restrict__ rows, int row_stride, int input_at, i
     float* maxima = batch.state + (size_t)batch.slot_ids[s] * batch.state_stride + batch.state_offset + head;      // (m_offset)
     if (threadIdx.x == 0) carried = p_first > 0 ? maxima[(size_t)((p_first - 1) & 1) * heads] : 0.0f;
     const float bi = input_bias[head], bf = forget_bias[head];
-    for (int t0 = 0; t0 < count; t0 += LS_THREADS * EG_EACH) {
+    for (int t0 = 0; t0 < count; t0 += EG_THREADS * EG_EACH) {
         float i[EG_EACH], f[EG_EACH];
         const int mine = t0 + threadIdx.x * EG_EACH;
         GateRun run = {0.0f, -INFINITY};
@@ -829,7 +829,7 @@ exp_gates_kernel(const float* __restrict__ rows, int row_stride, int input_at, i
             key_scale[at] = expf(i[e] - top);
             floor[at] = expf(-top);
             m = top;
-            if (mine + e == min(count, t0 + LS_THREADS * EG_EACH) - 1) {       // the last token of this round
+            if (mine + e == min(count, t0 + EG_THREADS * EG_EACH) - 1) {       // the last token of this round
                 carried = m;
                 if (mine + e == count - 1) maxima[(size_t)(p_last & 1) * heads] = m;
             }
@@ -1145,6 +1145,6 @@ SKV_EXPORT int skv_exp_gates(const float* rows, int row_stride, int input_at, in
         forget_at + heads > row_stride || m_offset < 0 || m_offset + 2LL * heads > state_stride)
         return fail(name, "the gates must lie inside a row and the maxima inside a slot's state");
     const LinearStateBatch batch = {positions, cu_q, slot_ids, state, state_stride, m_offset};
-    return launch_pdl(name, exp_gates_kernel, dim3(heads, n_seqs), dim3(LS_THREADS), 0, stream, rows, row_stride, input_at,
+    return launch_pdl(name, exp_gates_kernel, dim3(heads, n_seqs), dim3(EG_THREADS), 0, stream, rows, row_stride, input_at,
                       forget_at, input_bias, forget_bias, cap, log_decay, key_scale, floor, heads, batch);
 }
