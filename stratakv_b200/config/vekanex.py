@@ -13,8 +13,8 @@ The file names the design under ``architecture`` and lists its layers, each with
                   "left_scale": a, "right_scale": b}, "mlp": ...},
        {..., "weights_of": j}]}
 
-A layer with ``weights_of`` has no tensors of its own and uses layer j's; the rest of its entry equals layer j's.  Every size
-and every constant that differs between models of the design comes from there; sizes that only a tensor's shape gives (the
+``weights_of`` makes an entry one more run of layer j on that layer's tensors, with pages and state of its own; an entry that
+says otherwise about its mixer or feed-forward than layer j is refused.  Every size and every constant that differs between models of the design comes from there; sizes that only a tensor's shape gives (the
 ranks of the low-rank parts) are read from the checkpoint's header by the loader, or are given as ``mixer.rank`` (``gla``) and
 ``mixer.right.decay_rank`` and ``mixer.right.gate_rank`` (``parallel``).
 """

@@ -15,6 +15,7 @@
 
 namespace skv {
 
+constexpr int NR_THREADS = 256;
 
 struct NormedRotary {
     int heads, kv_heads, dim, vdim, q_width, v_width, row_stride;
@@ -30,8 +31,7 @@ struct NormedRotary {
     int write_kv;
 };
 
-// Sums of two numbers over the block; every thread gets both.  `scratch` holds two floats a warp.
-template <int NR_THREADS>
+// Sums of two numbers over the block; every thread gets both.  `scratch` holds 18 floats.
 __device__ __forceinline__ float2 block_sum2(float a, float b, float* scratch) {
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     a = warp_sum(a);
@@ -47,8 +47,7 @@ __device__ __forceinline__ float2 block_sum2(float a, float b, float* scratch) {
 // VEC: head sizes, widths and the row stride are multiples of 4, the rotation is interleaved (or absent, or its halves are
 // multiples of 4) and every pointer is 16-byte aligned: four neighbouring numbers (two pairs, or one side of four) a thread
 // and round.
-// NR_THREADS: 256 where a step has tokens enough to fill the GPU, else 1024.
-template <typename T, bool VEC, int NR_THREADS>
+template <typename T, bool VEC>
 __global__ void __launch_bounds__(NR_THREADS)
 normed_rotary_kernel(const float* __restrict__ rows, const int* __restrict__ positions, const int* __restrict__ token_seq,
                      const int* __restrict__ block_table, int table_width, T* __restrict__ q_out, T* __restrict__ k_cache,
@@ -95,7 +94,7 @@ normed_rotary_kernel(const float* __restrict__ rows, const int* __restrict__ pos
             if (a.q_weight) for (int i = threadIdx.x; i < nq; i += NR_THREADS) { const float x = load1(q, bq, i); sq = fmaf(x, x, sq); }
             if (a.k_weight) for (int i = threadIdx.x; i < nk; i += NR_THREADS) { const float x = load1(k, bk, i); sk = fmaf(x, x, sk); }
         }
-        const float2 sums = block_sum2<NR_THREADS>(sq, sk, scratch);
+        const float2 sums = block_sum2(sq, sk, scratch);
         if (a.q_weight) q_factor = 1.0f / sqrtf(sums.x / (float)nq + a.eps);
         if (a.k_weight) k_factor = 1.0f / sqrtf(sums.y / (float)nk + a.eps);
     }
@@ -236,9 +235,7 @@ SKV_EXPORT int skv_normed_rotary(const float* rows, int row_stride, const float*
     const bool vec = ((dim | vdim | q_width | v_width | row_stride) & 3) == 0 && (interleaved || rotated % 8 == 0) &&
                      (((uintptr_t)rows | (uintptr_t)bias | (uintptr_t)q_weight | (uintptr_t)k_weight | (uintptr_t)first | (uintptr_t)keep |
                        (uintptr_t)q_out | (uintptr_t)k_cache | (uintptr_t)v_cache) & 15) == 0;
-    const bool few = n <= 2 * sm_count() && heads * dim > 1024;
-    auto kernel = few ? (vec ? normed_rotary_kernel<skv_t, true, 1024> : normed_rotary_kernel<skv_t, false, 1024>)
-                      : (vec ? normed_rotary_kernel<skv_t, true, 256> : normed_rotary_kernel<skv_t, false, 256>);
-    return launch_pdl(name, kernel, dim3(n), dim3(few ? 1024 : 256), 0, stream, rows, positions, token_seq, block_table, table_width,
+    auto kernel = vec ? normed_rotary_kernel<skv_t, true> : normed_rotary_kernel<skv_t, false>;
+    return launch_pdl(name, kernel, dim3(n), dim3(NR_THREADS), 0, stream, rows, positions, token_seq, block_table, table_width,
                       (skv_t*)q_out, (skv_t*)k_cache, (skv_t*)v_cache, block_size, a);
 }

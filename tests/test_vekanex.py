@@ -264,7 +264,7 @@ def test_a_fault_moves_the_plain_logits_far_more_than_rounding(model_va, fault):
 
 
 def _read_first(q, k, v, beta, log_decay):
-    """The read-out misses the current token's write."""
+    """A token reads the state before it has written its own share."""
     T, H, n = k.shape
     S = torch.zeros(H, n, v.shape[2], dtype=F64)
     o = torch.zeros(T, H, v.shape[2], dtype=F64)
