@@ -14,9 +14,10 @@ The file names the design under ``architecture`` and lists its layers, each with
        {..., "weights_of": j}]}
 
 ``weights_of`` makes an entry one more run of layer j on that layer's tensors, with pages and state of its own; an entry that
-says otherwise about its mixer or feed-forward than layer j is refused.  Every size and every constant that differs between models of the design comes from there; sizes that only a tensor's shape gives (the
-ranks of the low-rank parts) are read from the checkpoint's header by the loader, or are given as ``mixer.rank`` (``gla``) and
-``mixer.right.decay_rank`` and ``mixer.right.gate_rank`` (``parallel``).
+says otherwise about its mixer or feed-forward than layer j is refused.  Every size and every constant that differs between
+models of the design comes from there; sizes that only a tensor's shape gives (the ranks of the low-rank parts) are read from
+the checkpoint's header by the loader, or are given as ``mixer.rank`` (``gla``) and ``mixer.right.decay_rank`` and
+``mixer.right.gate_rank`` (``parallel``).
 """
 from __future__ import annotations
 
